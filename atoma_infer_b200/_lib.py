@@ -197,7 +197,11 @@ class HybridLayer(C.Structure):
                 [(n, C.c_int64) for n in ("r_heads", "r_kv_heads", "r_dim", "r_vdim", "r_taps", "rq_off", "rk_off", "rv_off", "rg_off", "rb_off",
                                           "ra_off")] +
                 [(n, C.c_void_p) for n in ("r_tap_w", "r_a_log", "r_dt_bias", "r_head_norm", "r_w_o", "out_norm_a", "out_norm_b")] +
-                [("rot_dim", C.c_int64)])
+                [("rot_dim", C.c_int64)] +
+                # post-norm blocks: depth average, per-head score factors, rotation details, real-gated linear recurrent unit
+                [(n, C.c_void_p) for n in ("depth_w", "q_head_scale", "qk_freq_lo")] + [("rot_amplitude", C.c_float), ("route_group_top", C.c_int32)] +
+                [(n, C.c_int64) for n in ("lru_width", "lru_blocks")] +
+                [(n, C.c_void_p) for n in ("lru_w", "lru_bias_r", "lru_bias_i", "lru_rate", "r_tap_bias", "w_uk_rot")])
 
 
 class HybridModel(C.Structure):
@@ -209,7 +213,7 @@ class HybridModel(C.Structure):
                 [("layers", C.POINTER(HybridLayer))] +
                 [("block_style", C.c_int32), ("norm_groups", C.c_int32), ("pos_table", C.c_void_p), ("max_positions", C.c_int64),
                  ("logit_softcap", C.c_float), ("side_table", C.c_void_p), ("side_dim", C.c_int64), ("side_table_width", C.c_int64),
-                 ("lanes", C.c_int32), ("embed_scale", C.c_float)])
+                 ("lanes", C.c_int32), ("embed_scale", C.c_float), ("embed_norm", C.c_void_p), ("residual_alpha", C.c_float)])
 
 
 class GatedResidualArgs(C.Structure):
@@ -258,7 +262,7 @@ class TapFilterArgs(C.Structure):
                 [("ld_out", C.c_int64), ("history", C.c_void_p), ("history_stride", C.c_int64)] +
                 [(n, C.c_void_p) for n in ("state_slots", "token_seq", "query_start", "context_lens")] +
                 [(n, C.c_int64) for n in ("T", "B", "channels", "taps")] +
-                [("residual", C.c_int32), ("act", C.c_int32), ("dtype", C.c_uint32)])
+                [("residual", C.c_int32), ("act", C.c_int32), ("dtype", C.c_uint32), ("in_bias", C.c_void_p), ("bias1", C.c_void_p)])
 
 
 class StateScanArgs(C.Structure):
@@ -280,7 +284,32 @@ class QkvRopeArgs(C.Structure):
                 [(n, C.c_void_p) for n in ("q_weight", "k_weight", "qk_freq", "v_freq")] +
                 [("rot_pairs", C.c_int64), ("v_pairs", C.c_int64), ("interleaved", C.c_int32)] +
                 [(n, C.c_void_p) for n in ("positions", "slot_mapping", "q_out", "k_cache", "v_cache")] +
-                [(n, C.c_int64) for n in ("T", "H", "G", "dim", "vdim")] + [("eps", C.c_float), ("dtype", C.c_uint32)])
+                [(n, C.c_int64) for n in ("T", "H", "G", "dim", "vdim")] + [("eps", C.c_float), ("dtype", C.c_uint32), ("bias", C.c_void_p),
+                                                                          ("q_head_scale", C.c_void_p), ("unit_norm", C.c_int32)])
+
+
+class PostnormArgs(C.Structure):
+    """struct atoma_postnorm_args"""
+
+    _fields_ = ([(n, C.c_void_p) for n in ("y", "expert_out", "pair_row", "top_expert")] + [("top", C.c_int64)] +
+                [(n, C.c_void_p) for n in ("x", "w_norm", "depth", "depth_w")] + [("depth_n", C.c_int64), ("h", C.c_void_p), ("trace", C.c_void_p)] +
+                [("T", C.c_int64), ("width", C.c_int64), ("alpha", C.c_float), ("eps", C.c_float), ("weight_offset", C.c_float), ("dtype", C.c_uint32)])
+
+
+class LruGatesArgs(C.Structure):
+    """struct atoma_lru_gates_args"""
+
+    _fields_ = ([("u", C.c_void_p), ("ld_u", C.c_int64)] + [(n, C.c_void_p) for n in ("w", "bias_r", "bias_i", "rate", "decay", "input")] +
+                [(n, C.c_int64) for n in ("T", "channels", "blocks")] + [("dtype", C.c_uint32)])
+
+
+class LinearScanArgs(C.Structure):
+    """struct atoma_linear_scan_args"""
+
+    _fields_ = ([(n, C.c_void_p) for n in ("decay", "input", "gate")] + [("ld_gate", C.c_int64), ("gate_bias", C.c_void_p), ("state", C.c_void_p),
+                                                                          ("state_stride", C.c_int64)] +
+                [(n, C.c_void_p) for n in ("state_slots", "query_start", "context_lens", "out")] +
+                [(n, C.c_int64) for n in ("T", "B", "channels")] + [("act", C.c_int32), ("max_query_len", C.c_int32), ("dtype", C.c_uint32)])
 
 
 class LatentAttnArgs(C.Structure):
@@ -445,7 +474,7 @@ SIGNATURES = {
     "atoma_qk_headnorm_cache": (None, [C.c_void_p] + [C.c_int64] * 4 + [C.c_void_p, C.c_void_p, C.c_float] + [C.c_void_p] * 4 + [C.c_int64] * 5 +
                                 [C.c_float, C.c_uint32, C.c_void_p]),
     "atoma_softmax_attention_paged": (None, [C.POINTER(SoftmaxAttnArgs), C.c_void_p]),
-    "atoma_moe_route_grouped": (None, [C.c_void_p] * 5 + [C.c_int64] * 6 + [C.c_int32, C.c_int32, C.c_uint32, C.c_void_p]),
+    "atoma_moe_route_grouped": (None, [C.c_void_p] * 5 + [C.c_int64] * 6 + [C.c_int32] * 3 + [C.c_uint32, C.c_void_p]),
     "atoma_glu_clamped_bias": (None, [C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_int64, C.c_int64, C.c_float, C.c_float, C.c_float,
                                       C.c_uint32, C.c_void_p]),
     "atoma_linear_glu_clamped": (None, [C.c_void_p] * 5 + [C.c_int64] * 3 + [C.c_float] * 3 + [C.c_uint32, C.c_void_p]),
@@ -455,11 +484,14 @@ SIGNATURES = {
     "atoma_headnorm_gate": (None, [C.c_void_p] * 3 + [C.c_int64, C.c_void_p] + [C.c_int64] * 3 + [C.c_float, C.c_uint32, C.c_void_p]),
     "atoma_qkv_headnorm_rope_cache": (None, [C.POINTER(QkvRopeArgs), C.c_void_p]),
     "atoma_rotate_heads": (None, [C.c_void_p] * 3 + [C.c_int64] * 4 + [C.c_int32, C.c_float, C.c_uint32, C.c_void_p]),
-    "atoma_latent_norm_rope_cache": (None, [C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int64, C.c_int32] + [C.c_void_p] * 4 +
+    "atoma_latent_norm_rope_cache": (None, [C.c_void_p, C.c_int64] + [C.c_void_p] * 4 + [C.c_float, C.c_int64, C.c_int32] + [C.c_void_p] * 4 +
                                      [C.c_int64] * 4 + [C.c_float, C.c_uint32, C.c_void_p]),
-    "atoma_latent_query_absorb_rope": (None, [C.c_void_p, C.c_void_p, C.c_void_p, C.c_int64, C.c_int32, C.c_void_p, C.c_void_p] + [C.c_int64] * 5 +
+    "atoma_latent_query_absorb_rope": (None, [C.c_void_p] * 4 + [C.c_float, C.c_int64, C.c_int32, C.c_void_p, C.c_void_p] + [C.c_int64] * 5 +
                                        [C.c_uint32, C.c_void_p]),
-    "atoma_latent_expand_values": (None, [C.c_void_p] * 3 + [C.c_int64] * 5 + [C.c_uint32, C.c_void_p]),
+    "atoma_latent_expand_values": (None, [C.c_void_p] * 3 + [C.c_int64, C.c_void_p] + [C.c_int64] * 5 + [C.c_uint32, C.c_void_p]),
+    "atoma_postnorm_residual": (None, [C.POINTER(PostnormArgs), C.c_void_p]),
+    "atoma_lru_gates": (None, [C.POINTER(LruGatesArgs), C.c_void_p]),
+    "atoma_linear_scan": (None, [C.POINTER(LinearScanArgs), C.c_void_p]),
     "atoma_hybrid_abi_sizeof": (C.c_int64, [C.c_int]),
     "atoma_hybrid_scratch_bytes": (C.c_int64, [C.POINTER(HybridModel), C.c_int64, C.c_int64]),
     "atoma_hybrid_step": (None, [C.POINTER(HybridModel), C.POINTER(HybridBatch), C.c_void_p]),

@@ -351,6 +351,7 @@ __global__ void __launch_bounds__(32 * kScanSeg) mingru_scan_kernel(const T *__r
     float *st = state + (live ? static_cast<int64_t>(slots[b]) * S + c : 0);
     float s = (live && context_lens[b] > 0) ? *st : 0.f;
     for (int k = 0; k < seg; ++k) s = sa[k][lane] * s + sb[k][lane];
+    __syncthreads();          // every row has read the carried state before the last one replaces it
     if (!live) return;
     for (int t = lo; t < hi; t += kBatch) {
         T zr[kBatch], ur[kBatch], gr[kBatch];

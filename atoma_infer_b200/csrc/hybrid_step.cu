@@ -50,7 +50,7 @@ bool hyb_latent_attention_expanded(const atoma_latent_expanded_args &, cudaStrea
 bool hyb_moe_route(const void *, const float *, const float *, int32_t *, float *, float *, int64_t, int64_t, int64_t, int64_t, int32_t,
                    uint32_t, cudaStream_t);
 bool hyb_moe_route_grouped(const void *, const float *, const float *, int32_t *, float *, int64_t, int64_t, int64_t, int64_t, int64_t, int64_t,
-                           int32_t, int32_t, uint32_t, cudaStream_t);
+                           int32_t, int32_t, int32_t, uint32_t, cudaStream_t);
 bool hyb_embed_scaled_lanes(const uint32_t *, const void *, float, float *, int64_t, int64_t, int64_t, int64_t, uint32_t, cudaStream_t);
 bool hyb_lanes_read_norm(const float *, const float *, const int32_t *, const float *, float, void *, float *, int64_t, int64_t, int64_t, float,
                          uint32_t, cudaStream_t);
@@ -67,11 +67,14 @@ bool hyb_state_scan(const atoma_state_scan_args &, cudaStream_t);
 bool hyb_headnorm_gate(const float *, const float *, const void *, int64_t, void *, int64_t, int64_t, int64_t, float, uint32_t, cudaStream_t);
 bool hyb_qkv_headnorm_rope_cache(const atoma_qkv_rope_args &, cudaStream_t);
 bool hyb_rotate_heads(void *, const int64_t *, const float *, int64_t, int64_t, int64_t, int64_t, int32_t, float, uint32_t, cudaStream_t);
-bool hyb_latent_norm_rope_cache(const void *, int64_t, const float *, const float *, const float *, int64_t, int32_t, const int64_t *,
-                                const int64_t *, void *, void *, int64_t, int64_t, int64_t, int64_t, float, uint32_t, cudaStream_t);
-bool hyb_latent_query_absorb_rope(const void *, const void *, const float *, int64_t, int32_t, const int64_t *, float *, int64_t, int64_t, int64_t,
-                                  int64_t, int64_t, uint32_t, cudaStream_t);
-bool hyb_latent_expand_values(const float *, const void *, void *, int64_t, int64_t, int64_t, int64_t, int64_t, uint32_t, cudaStream_t);
+bool hyb_latent_norm_rope_cache(const void *, int64_t, const float *, const float *, const float *, const float *, float, int64_t, int32_t,
+                                const int64_t *, const int64_t *, void *, void *, int64_t, int64_t, int64_t, int64_t, float, uint32_t, cudaStream_t);
+bool hyb_latent_query_absorb_rope(const void *, const void *, const float *, const float *, float, int64_t, int32_t, const int64_t *, float *, int64_t,
+                                  int64_t, int64_t, int64_t, int64_t, uint32_t, cudaStream_t);
+bool hyb_postnorm_residual(const atoma_postnorm_args &, cudaStream_t);
+bool hyb_lru_gates(const atoma_lru_gates_args &, cudaStream_t);
+bool hyb_linear_scan(const atoma_linear_scan_args &, cudaStream_t);
+bool hyb_latent_expand_values(const float *, const void *, const void *, int64_t, void *, int64_t, int64_t, int64_t, int64_t, int64_t, uint32_t, cudaStream_t);
 int64_t hyb_moe_workspace_bytes(int64_t, int64_t, int64_t, int64_t, int64_t, uint32_t);
 bool hyb_moe_experts(const atoma_moe_args &, const void **, const int32_t **, cudaStream_t);
 
@@ -85,6 +88,8 @@ struct Widths {
     int64_t moe = 0;                    // bytes of the routed experts' workspace
     int64_t conv = 0, of32 = 0;         // parallel blocks: filtered q / k / v row of a delta-rule mixer, float32 read-out row of a recurrence
     bool parallel = false, keep_embedding = false;
+    int64_t lru = 0;                    // post-norm blocks: channels of a linear recurrent unit
+    int64_t depth = 0;                  // float32 [T, width] planes of the average over depth
 };
 
 inline bool gated(const float *bias) { return bias != nullptr; }
@@ -98,6 +103,32 @@ Widths widths(const atoma_hybrid_model &m, int64_t T) {
     Widths w;
     for (int64_t i = 0; i < m.num_layers; ++i) {
         const atoma_hybrid_layer &l = m.layers[i];
+        if (m.block_style == ATOMA_BLOCK_POSTNORM) {
+            if (l.depth_w) w.depth = m.num_layers + 1;
+            w.proj = std::max(w.proj, l.proj_cols);
+            if (l.mixer == ATOMA_MIXER_SOFTMAX_ATTENTION) {
+                w.q = std::max(w.q, l.heads * l.dim);
+                w.act = std::max(w.act, l.heads * l.vdim);
+            } else if (l.mixer == ATOMA_MIXER_LATENT_ATTENTION) {
+                w.q = std::max(w.q, l.heads * (l.dim + l.rot_dim));
+                w.cq = std::max(w.cq, l.q_rank);
+                w.act = std::max(w.act, l.heads * l.vdim);
+                w.lat = std::max(w.lat, l.heads * (l.kv_rank + l.rot_dim));
+            } else if (l.mixer == ATOMA_MIXER_LRU) {
+                w.act = std::max(w.act, l.lru_width);
+                w.conv = std::max(w.conv, l.lru_width);
+                w.lru = std::max(w.lru, l.lru_width);
+            }
+            if (l.has_mlp) {
+                w.proj = std::max(w.proj, 2 * l.ff);
+                w.act = std::max(w.act, l.ff);
+                if (l.ff_kind == ATOMA_FF_MOE) {
+                    w.route = std::max(w.route, l.top);
+                    w.moe = std::max(w.moe, hyb_moe_workspace_bytes(T, l.top, l.experts, m.width, l.expert_ff, m.dtype));
+                }
+            }
+            continue;
+        }
         if (m.block_style == ATOMA_BLOCK_PARALLEL) {
             w.parallel = true;
             w.keep_embedding = w.keep_embedding || l.add_embedding;
@@ -182,6 +213,8 @@ struct Scratch {
     // parallel blocks
     float *x0, *of32;
     char *h1, *h2, *y2, *yf, *conv;
+    // post-norm blocks
+    float *depth, *decay, *input;
     int64_t total;
 };
 
@@ -222,6 +255,9 @@ Scratch carve(const atoma_hybrid_model &m, int64_t T, int64_t S, void *base) {
     s.y2 = take(w.parallel ? T * m.width * es : 0);
     s.yf = take(w.parallel ? T * m.width * es : 0);
     s.conv = take(T * w.conv * es);
+    s.depth = reinterpret_cast<float *>(take(w.depth * T * m.width * 4));
+    s.decay = reinterpret_cast<float *>(take(T * w.lru * 4));
+    s.input = reinterpret_cast<float *>(take(T * w.lru * 4));
     s.total = off;
     return s;
 }
@@ -495,7 +531,7 @@ bool lanes_layer(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, const
     if (l.ff_kind == ATOMA_FF_MOE) {
         const int64_t outputs = l.experts + l.identity_experts;
         if (!hyb_moe_route_grouped(s.h, l.w_router, l.router_correction, s.top_expert, s.top_weight, T, W, outputs, l.top, l.route_groups,
-                                   l.route_keep, l.score_fn, l.renormalize, dt, stream))
+                                   l.route_keep, l.route_group_top, l.score_fn, l.renormalize, dt, stream))
             return false;
         atoma_moe_args e{};
         e.h = s.h;
@@ -614,12 +650,12 @@ bool parallel_layer(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, co
         r.y_a = s.y;
     } else if (l.mixer == ATOMA_MIXER_LATENT_ATTENTION) {
         const int64_t H = l.heads, row = l.kv_rank + l.rot_dim;
-        if (!hyb_latent_norm_rope_cache(s.proj, P, l.dq_norm, l.dkv_norm, l.qk_freq, l.rot_pairs, l.rot_interleaved, b.positions, b.slot_mapping,
-                                        s.cq, l.latent_cache, T, l.q_rank, l.kv_rank, l.rot_dim, m.eps, dt, stream))
+        if (!hyb_latent_norm_rope_cache(s.proj, P, l.dq_norm, l.dkv_norm, l.qk_freq, nullptr, 1.f, l.rot_pairs, l.rot_interleaved, b.positions,
+                                        b.slot_mapping, s.cq, l.latent_cache, T, l.q_rank, l.kv_rank, l.rot_dim, m.eps, dt, stream))
             return false;
         if (!hyb_linear(s.cq, l.w_uq, s.q, T, H * (l.dim + l.rot_dim), l.q_rank, dt, stream)) return false;
-        if (!hyb_latent_query_absorb_rope(s.q, l.w_uk, l.qk_freq, l.rot_pairs, l.rot_interleaved, b.positions, s.qlat, T, H, l.dim, l.rot_dim,
-                                          l.kv_rank, dt, stream))
+        if (!hyb_latent_query_absorb_rope(s.q, l.w_uk, l.qk_freq, nullptr, 1.f, l.rot_pairs, l.rot_interleaved, b.positions, s.qlat, T, H, l.dim,
+                                          l.rot_dim, l.kv_rank, dt, stream))
             return false;
         atoma_latent_attn_args a{};
         a.q_lat = s.qlat;
@@ -643,7 +679,7 @@ bool parallel_layer(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, co
         a.max_seq_len = b.max_seq_len;
         a.out_cols = l.kv_rank;            // the rotated tail of a cached row takes part in the scores only
         if (!hyb_latent_attention(a, stream)) return false;
-        if (!hyb_latent_expand_values(s.olat, l.w_uv, s.act, T, H, l.vdim, l.kv_rank, row, dt, stream)) return false;
+        if (!hyb_latent_expand_values(s.olat, l.w_uv, nullptr, 0, s.act, T, H, l.vdim, l.kv_rank, row, dt, stream)) return false;
         if (!hyb_linear(s.act, l.w_o, s.y, T, W, H * l.vdim, dt, stream)) return false;
         r.y_a = s.y;
     } else if (l.mixer == ATOMA_MIXER_PAIR) {
@@ -780,6 +816,244 @@ bool parallel_layer(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, co
     return hyb_parallel_residual_norm(r, stream);
 }
 
+// Softmax attention of a post-norm layer: stacked projection -> biases, unit norms, per-head factor, cache write -> attention -> s.act.
+bool postnorm_softmax(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, const atoma_hybrid_layer &l, const Scratch &s,
+                      cudaStream_t stream) {
+    atoma_qkv_rope_args q{};
+    q.proj = s.proj;
+    q.ld = l.proj_cols;
+    q.q_off = l.q_off;
+    q.k_off = l.k_off;
+    q.v_off = l.v_off;
+    q.positions = b.positions;
+    q.slot_mapping = b.slot_mapping;
+    q.q_out = s.q;
+    q.k_cache = l.k_cache;
+    q.v_cache = l.v_cache;
+    q.T = b.num_tokens;
+    q.H = l.heads;
+    q.G = l.kv_heads;
+    q.dim = l.dim;
+    q.vdim = l.vdim;
+    q.eps = m.eps;
+    q.dtype = m.dtype;
+    q.bias = l.b_qkv;
+    q.q_head_scale = l.q_head_scale;
+    q.unit_norm = 1;
+    if (!hyb_qkv_headnorm_rope_cache(q, stream)) return false;
+    atoma_softmax_attn_args a{};
+    a.q = s.q;
+    a.k_cache = l.k_cache;
+    a.v_cache = l.v_cache;
+    a.out = s.act;
+    a.positions = b.positions;
+    a.token_seq = b.token_seq;
+    a.query_start = b.query_start;
+    a.block_tables = b.block_tables;
+    a.T = b.num_tokens;
+    a.B = b.num_seqs;
+    a.max_blocks = b.max_blocks;
+    a.H = l.heads;
+    a.G = l.kv_heads;
+    a.dim = l.dim;
+    a.vdim = l.vdim;
+    a.block_size = m.block_size;
+    a.window = l.window;
+    a.scale = l.scale;
+    a.dtype = m.dtype;
+    a.max_query_len = b.max_query_len;
+    a.max_seq_len = b.max_seq_len;
+    a.long_min_q = b.long_min_q;
+    a.long_seqs = b.long_seqs;
+    a.long_tokens = b.long_tokens;
+    a.long_ctx_sum = b.long_ctx_sum;
+    return hyb_softmax_attention(a, stream);
+}
+
+// Latent attention of a post-norm layer: norms, rotation and cache write -> queries into the space of the cached rows -> attention
+// over them -> values (times the output gate) -> s.act.
+bool postnorm_latent(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, const atoma_hybrid_layer &l, const Scratch &s,
+                     cudaStream_t stream) {
+    const uint32_t dt = m.dtype;
+    const int64_t es = dt == ATOMA_DTYPE_F32 ? 4 : 2;
+    const int64_t T = b.num_tokens, H = l.heads, row = l.kv_rank + l.rot_dim, P = l.proj_cols;
+    const void *gate = l.out_gate ? s.proj + l.g_off * es : nullptr;
+    if (!hyb_latent_norm_rope_cache(s.proj, P, l.dq_norm, l.dkv_norm, l.qk_freq, l.qk_freq_lo, l.rot_amplitude, l.rot_pairs, l.rot_interleaved,
+                                    b.positions, b.slot_mapping, s.cq, l.latent_cache, T, l.q_rank, l.kv_rank, l.rot_dim, m.eps, dt, stream))
+        return false;
+    if (!hyb_linear(s.cq, l.w_uq, s.q, T, H * (l.dim + l.rot_dim), l.q_rank, dt, stream)) return false;
+    if (!hyb_latent_query_absorb_rope(s.q, l.w_uk, l.qk_freq, l.qk_freq_lo, l.rot_amplitude, l.rot_pairs, l.rot_interleaved, b.positions, s.qlat,
+                                      T, H, l.dim, l.rot_dim, l.kv_rank, dt, stream))
+        return false;
+    atoma_latent_attn_args a{};
+    a.q_lat = s.qlat;
+    a.latent_cache = l.latent_cache;
+    a.out = s.olat;
+    a.positions = b.positions;
+    a.token_seq = b.token_seq;
+    a.query_start = b.query_start;
+    a.block_tables = b.block_tables;
+    a.sink = l.sink;
+    a.T = T;
+    a.B = b.num_seqs;
+    a.max_blocks = b.max_blocks;
+    a.H = H;
+    a.R = row;
+    a.block_size = m.block_size;
+    a.window = l.window;
+    a.scale = l.scale;
+    a.dtype = dt;
+    a.max_query_len = b.max_query_len;
+    a.max_seq_len = b.max_seq_len;
+    a.out_cols = l.kv_rank;            // the rotated tail of a cached row takes part in the scores only
+    if (!hyb_latent_attention(a, stream)) return false;
+    return hyb_latent_expand_values(s.olat, l.w_uv, gate, P, s.act, T, H, l.vdim, l.kv_rank, row, dt, stream);
+}
+
+// Recurrent block of a post-norm layer: short filter -> gates -> scan, times the activated gate branch -> s.act.
+bool postnorm_lru(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, const atoma_hybrid_layer &l, const Scratch &s, cudaStream_t stream) {
+    const uint32_t dt = m.dtype;
+    const int64_t es = dt == ATOMA_DTYPE_F32 ? 4 : 2;
+    const int64_t C = l.lru_width, hist = l.r_taps > 1 ? (l.r_taps - 1) * C : 0;
+    if (!l.layer_state) {
+        set_status(kErrInvalidArg, "atoma_hybrid_step: a recurrent layer has no state");
+        return false;
+    }
+    atoma_tap_filter_args f{};
+    f.in = s.proj + l.k_off * es;
+    f.ld_in = l.proj_cols;
+    f.w1 = l.r_tap_w;
+    f.out1 = s.conv;
+    f.ld_out = C;
+    f.history = l.layer_state;
+    f.history_stride = l.layer_state_stride;
+    f.state_slots = b.state_slots;
+    f.token_seq = b.token_seq;
+    f.query_start = b.query_start;
+    f.context_lens = b.context_lens;
+    f.T = b.num_tokens;
+    f.B = b.num_seqs;
+    f.channels = C;
+    f.taps = l.r_taps;
+    f.dtype = dt;
+    f.in_bias = l.b_qkv ? l.b_qkv + l.k_off : nullptr;
+    f.bias1 = l.r_tap_bias;
+    if (!hyb_tap_filter(f, stream)) return false;
+    atoma_lru_gates_args g{};
+    g.u = s.conv;
+    g.ld_u = C;
+    g.w = l.lru_w;
+    g.bias_r = l.lru_bias_r;
+    g.bias_i = l.lru_bias_i;
+    g.rate = l.lru_rate;
+    g.decay = s.decay;
+    g.input = s.input;
+    g.T = b.num_tokens;
+    g.channels = C;
+    g.blocks = l.lru_blocks;
+    g.dtype = dt;
+    if (!hyb_lru_gates(g, stream)) return false;
+    atoma_linear_scan_args a{};
+    a.decay = s.decay;
+    a.input = s.input;
+    a.gate = s.proj + l.q_off * es;
+    a.ld_gate = l.proj_cols;
+    a.gate_bias = l.b_qkv ? l.b_qkv + l.q_off : nullptr;
+    a.state = l.layer_state + hist;
+    a.state_stride = l.layer_state_stride;
+    a.state_slots = b.state_slots;
+    a.query_start = b.query_start;
+    a.context_lens = b.context_lens;
+    a.out = s.act;
+    a.T = b.num_tokens;
+    a.B = b.num_seqs;
+    a.channels = C;
+    a.act = l.act;
+    a.max_query_len = b.max_query_len;
+    a.dtype = dt;
+    return hyb_linear_scan(a, stream);
+}
+
+// One layer of a post-norm design: x <- norm1(alpha x + mixer(x)); x <- norm2(alpha x + ff(x)); then the average over depth.  s.h holds
+// x in the activation format on entry and the next layer's on return; the stream itself is s.x.
+bool postnorm_layer(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, const atoma_hybrid_layer &l, int64_t index, const Scratch &s,
+                    float *trace, cudaStream_t stream) {
+    const uint32_t dt = m.dtype;
+    const int64_t T = b.num_tokens, W = m.width;
+    if (!hyb_linear(s.h, l.w_qkv, s.proj, T, l.proj_cols, W, dt, stream)) return false;
+    int64_t mixed = l.heads * l.vdim;
+    if (l.mixer == ATOMA_MIXER_SOFTMAX_ATTENTION) {
+        if (!postnorm_softmax(m, b, l, s, stream)) return false;
+    } else if (l.mixer == ATOMA_MIXER_LATENT_ATTENTION) {
+        if (!postnorm_latent(m, b, l, s, stream)) return false;
+    } else if (l.mixer == ATOMA_MIXER_LRU) {
+        if (!postnorm_lru(m, b, l, s, stream)) return false;
+        mixed = l.lru_width;
+    } else {
+        set_status(kErrUnsupported, "atoma_hybrid_step: post-norm layers take softmax attention, latent attention or the linear recurrent unit, got %d",
+                   l.mixer);
+        return false;
+    }
+    if (!hyb_linear(s.act, l.w_o, s.y, T, W, mixed, dt, stream)) return false;
+    atoma_postnorm_args r{};
+    r.y = s.y;
+    r.x = s.x;
+    r.w_norm = l.norm1;
+    r.h = s.h;
+    r.T = T;
+    r.width = W;
+    r.alpha = m.residual_alpha;
+    r.eps = m.eps;
+    r.weight_offset = m.norm_offset;
+    r.dtype = dt;
+    atoma_postnorm_args f = r;          // the layer's last update
+    f.w_norm = l.has_mlp ? l.norm2 : l.norm1;
+    f.depth = l.depth_w ? s.depth : nullptr;
+    f.depth_w = l.depth_w;
+    f.depth_n = l.depth_w ? index + 2 : 0;
+    f.trace = trace;
+    if (!l.has_mlp) return hyb_postnorm_residual(f, stream);
+    if (!hyb_postnorm_residual(r, stream)) return false;
+    f.y = nullptr;
+    const bool moe = l.ff_kind == ATOMA_FF_MOE;
+    if (l.ff > 0) {   // the dense feed-forward, or the shared expert of a mixture
+        if (!hyb_gate_up_act(s.h, moe ? l.w_ff_in : l.w_gate_up, s.proj, s.act, T, l.ff, W, ATOMA_ACT_SILU, dt, stream)) return false;
+        if (!hyb_linear(s.act, l.w_down, s.y, T, W, l.ff, dt, stream)) return false;
+        f.y = s.y;
+    }
+    if (moe) {
+        if (!hyb_moe_route_grouped(s.h, l.w_router, l.router_correction, s.top_expert, s.top_weight, T, W, l.experts, l.top, l.route_groups,
+                                   l.route_keep, l.route_group_top, l.score_fn, l.renormalize, dt, stream))
+            return false;
+        atoma_moe_args e{};
+        e.h = s.h;
+        e.top_expert = s.top_expert;
+        e.top_weight = s.top_weight;
+        e.w_gate_up = l.w_expert_gate_up;
+        e.w_down = l.w_expert_down;
+        e.workspace = s.moe;
+        e.workspace_bytes = s.moe_bytes;
+        e.T = T;
+        e.width = W;
+        e.experts = l.experts;
+        e.top = l.top;
+        e.ff = l.expert_ff;
+        e.limit = l.expert_limit;
+        e.alpha = l.act_alpha;   // alpha 1, shift 0, no limit: silu(gate) * up
+        e.up_shift = l.act_up_shift;
+        e.scale_input = l.scale_input;
+        e.dtype = dt;
+        const void *eo = nullptr;
+        const int32_t *pr = nullptr;
+        if (!hyb_moe_experts(e, &eo, &pr, stream)) return false;
+        f.expert_out = eo;
+        f.pair_row = pr;
+        f.top_expert = s.top_expert;
+        f.top = l.top;
+    }
+    return hyb_postnorm_residual(f, stream);
+}
+
 }  // namespace
 }  // namespace atoma
 
@@ -801,6 +1075,9 @@ extern "C" int64_t atoma_hybrid_abi_sizeof(int which) {
         case 11: return sizeof(atoma_tap_filter_args);
         case 12: return sizeof(atoma_state_scan_args);
         case 13: return sizeof(atoma_qkv_rope_args);
+        case 14: return sizeof(atoma_postnorm_args);
+        case 15: return sizeof(atoma_lru_gates_args);
+        case 16: return sizeof(atoma_linear_scan_args);
         default: return -1;
     }
 }
@@ -822,7 +1099,8 @@ extern "C" void atoma_hybrid_step(const atoma_hybrid_model *model, const atoma_h
     const int64_t T = b.num_tokens, B = b.num_seqs, S = b.num_selected;
     if (T <= 0 || B <= 0) return;
     if (!b.tokens || !b.positions || !b.slot_mapping || !b.token_seq || !b.query_start || !b.context_lens || !b.block_tables ||
-        !b.state_slots || !b.scratch || (S > 0 && (!b.selected || !b.logits)) || !m.embed || (!m.inv_freq && !m.pos_table && m.block_style != ATOMA_BLOCK_LANES && m.block_style != ATOMA_BLOCK_PARALLEL) || !m.final_norm ||
+        !b.state_slots || !b.scratch || (S > 0 && (!b.selected || !b.logits)) || !m.embed || (!m.inv_freq && !m.pos_table && m.block_style != ATOMA_BLOCK_LANES && m.block_style != ATOMA_BLOCK_PARALLEL &&
+          m.block_style != ATOMA_BLOCK_POSTNORM) || !m.final_norm ||
         !m.head || m.width <= 0 || m.vocab <= 0 || m.num_layers <= 0) {
         set_status(kErrInvalidArg, "atoma_hybrid_step: a required tensor is NULL");
         return;
@@ -841,6 +1119,36 @@ extern "C" void atoma_hybrid_step(const atoma_hybrid_model *model, const atoma_h
     const int64_t W = m.width;
     const float off = m.norm_offset;
     const int64_t groups = m.norm_groups > 0 ? m.norm_groups : 1;
+    if (m.block_style == ATOMA_BLOCK_POSTNORM) {
+        // the normed embedding rows are the first row of the average over depth
+        if (!m.embed_norm) {
+            set_status(kErrInvalidArg, "atoma_hybrid_step: a post-norm design needs the norm of the embedding");
+            return;
+        }
+        if (!hyb_embed_scaled_lanes(b.tokens, m.embed, 1.f, s.x, T, 1, W, m.vocab, dt, stream)) return;
+        atoma_postnorm_args r{};
+        r.x = s.x;
+        r.w_norm = m.embed_norm;
+        r.depth = m.layers[0].depth_w ? s.depth : nullptr;
+        r.depth_n = r.depth ? 1 : 0;
+        r.h = s.h;
+        r.T = T;
+        r.width = W;
+        r.alpha = 1.f;
+        r.eps = m.eps;
+        r.weight_offset = off;
+        r.dtype = dt;
+        if (!hyb_postnorm_residual(r, stream)) return;
+        for (int64_t i = 0; i < m.num_layers; ++i) {
+            if (!postnorm_layer(m, b, m.layers[i], i, s, b.residual_trace ? b.residual_trace + i * T * W : nullptr, stream)) return;
+        }
+        if (S > 0) {
+            if (!hyb_group_rmsnorm_rows(s.x, b.selected, m.final_norm, off, 1, s.hs, S, W, m.eps, dt, stream)) return;
+            if (!hyb_linear(s.hs, m.head, s.lg, S, m.vocab, W, dt, stream)) return;
+            if (!hyb_scale_greedy(s.lg, b.logits, b.next_tokens, S, m.vocab, m.logit_scale, m.logit_softcap, dt, stream)) return;
+        }
+        return;
+    }
     if (m.block_style == ATOMA_BLOCK_PARALLEL) {
         // the embedding rows (kept when a later pass adds them again), what precedes the first layer, its input norm
         const atoma_hybrid_layer &first = m.layers[0];

@@ -68,7 +68,8 @@ __global__ void __launch_bounds__(kRowThreads) latent_norm_cache_kernel(const T 
 template <typename TA, typename TW, typename TO>
 __global__ void __launch_bounds__(256) head_project_kernel(const TA *__restrict__ in, int64_t ld_in, int64_t in_hs,
                                                            const TW *__restrict__ w, int64_t w_hs, int64_t w_ks, int64_t w_ns,
-                                                           TO *__restrict__ out, int64_t ld_out, int64_t out_hs, int M, int N, int K) {
+                                                           TO *__restrict__ out, int64_t ld_out, int64_t out_hs, int M, int N, int K,
+                                                           const TO *__restrict__ gate, int64_t ld_gate) {
     __shared__ float xs[16][65], ws[16][65];
     pdl_launch_dependents();
     pdl_wait();
@@ -116,7 +117,10 @@ __global__ void __launch_bounds__(256) head_project_kernel(const TA *__restrict_
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
-            if (m < M && n < N) out[static_cast<int64_t>(m) * ld_out + n] = from_f<TO>(acc[i][j]);
+            if (m >= M || n >= N) continue;
+            float v = acc[i][j];
+            if (gate) v *= sigmoidf_(to_f(gate[static_cast<int64_t>(m) * ld_gate + h * out_hs + n]));
+            out[static_cast<int64_t>(m) * ld_out + n] = from_f<TO>(v);
         }
 }
 
@@ -589,12 +593,13 @@ bool hyb_latent_norm_cache(const void *proj, int64_t ld, const float *q_w, const
 
 // Per-head projection with explicit strides: head h of `in` starts in_hs elements into a row of ld_in, head h of `out`
 // out_hs elements into a row of ld_out (so heads that carry more than the projected part, or an output row that keeps
-// room for more, need no copies).  w [H n, R] as in atoma_head_project.
+// room for more, need no copies).  w [H n, R] as in atoma_head_project.  gate (absorb = 0 only, NULL: none; row stride ld_gate, the
+// result's number format): out times sigmoid(gate[t, h out_hs + j]).
 bool hyb_head_project_ld(const void *in, int64_t ld_in, int64_t in_hs, const void *w, void *out, int64_t ld_out, int64_t out_hs, int64_t T,
-                         int64_t H, int64_t n, int64_t R, int32_t absorb, uint32_t dtype, cudaStream_t stream) {
+                         int64_t H, int64_t n, int64_t R, int32_t absorb, uint32_t dtype, cudaStream_t stream, const void *gate, int64_t ld_gate) {
     if (T <= 0) return true;
     if (!hybrid::known_dtype(dtype, "atoma_head_project")) return false;
-    if (!in || !w || !out || H <= 0 || n <= 0 || R <= 0) {
+    if (!in || !w || !out || H <= 0 || n <= 0 || R <= 0 || (gate && absorb)) {
         set_status(kErrInvalidArg, "atoma_head_project: null argument or empty head");
         return false;
     }
@@ -614,6 +619,7 @@ bool hyb_head_project_ld(const void *in, int64_t ld_in, int64_t in_hs, const voi
             e = launch_ex(tc::gemm_kernel<__nv_bfloat16, float, false>, grid, dim3(128), 0, stream, p);
         } else {
             p.b_ks = 1, p.b_ns = R, p.N = static_cast<int>(n), p.K = static_cast<int>(R);
+            p.gate = static_cast<const __nv_bfloat16 *>(gate), p.ld_gate = ld_gate;
             const dim3 grid(static_cast<unsigned>((n + 63) / 64), static_cast<unsigned>((T + 63) / 64), static_cast<unsigned>(H));
             e = launch_ex(tc::gemm_kernel<float, __nv_bfloat16, false>, grid, dim3(128), 0, stream, p);
         }
@@ -623,14 +629,14 @@ bool hyb_head_project_ld(const void *in, int64_t ld_in, int64_t in_hs, const voi
         const dim3 grid(static_cast<unsigned>((R + 63) / 64), static_cast<unsigned>((T + 63) / 64), static_cast<unsigned>(H));
 #define CALL(TT) launch_ex(head_project_kernel<TT, TT, float>, grid, dim3(256), 0, stream, static_cast<const TT *>(in), ld_in, in_hs, \
                            static_cast<const TT *>(w), n * R, R, static_cast<int64_t>(1), static_cast<float *>(out), ld_out, out_hs, M, \
-                           static_cast<int>(R), static_cast<int>(n))
+                           static_cast<int>(R), static_cast<int>(n), static_cast<const float *>(nullptr), static_cast<int64_t>(0))
         e = HYB_DISPATCH(dtype, CALL);
 #undef CALL
     } else {
         const dim3 grid(static_cast<unsigned>((n + 63) / 64), static_cast<unsigned>((T + 63) / 64), static_cast<unsigned>(H));
 #define CALL(TT) launch_ex(head_project_kernel<float, TT, TT>, grid, dim3(256), 0, stream, static_cast<const float *>(in), ld_in, in_hs, \
                            static_cast<const TT *>(w), n * R, static_cast<int64_t>(1), R, static_cast<TT *>(out), ld_out, out_hs, M, \
-                           static_cast<int>(n), static_cast<int>(R))
+                           static_cast<int>(n), static_cast<int>(R), static_cast<const TT *>(gate), ld_gate)
         e = HYB_DISPATCH(dtype, CALL);
 #undef CALL
     }
@@ -639,8 +645,8 @@ bool hyb_head_project_ld(const void *in, int64_t ld_in, int64_t in_hs, const voi
 
 bool hyb_head_project(const void *in, const void *w, void *out, int64_t T, int64_t H, int64_t n, int64_t R, int32_t absorb, uint32_t dtype,
                       cudaStream_t stream) {
-    if (absorb) return hyb_head_project_ld(in, H * n, n, w, out, H * R, R, T, H, n, R, 1, dtype, stream);
-    return hyb_head_project_ld(in, H * R, R, w, out, H * n, n, T, H, n, R, 0, dtype, stream);
+    if (absorb) return hyb_head_project_ld(in, H * n, n, w, out, H * R, R, T, H, n, R, 1, dtype, stream, nullptr, 0);
+    return hyb_head_project_ld(in, H * R, R, w, out, H * n, n, T, H, n, R, 0, dtype, stream, nullptr, 0);
 }
 
 // The tensor-core kernel takes bfloat16 caches whose rows are a multiple of 64 entries (16-byte rows for cp.async, whole ldmatrix

@@ -169,12 +169,13 @@ __global__ void __launch_bounds__(128) moe_topk_kernel(const float *__restrict__
 
 // Router with a restricted choice: one warp per token over the float32 logits of all router outputs.
 // s = softmax or sigmoid of the logits; c = s + correction; the outputs form `groups` equal groups of neighbours, a group's
-// score is its largest c, only the `keep` best groups (ties: the lower group) can be chosen from; `top` rounds of arg-max of c
+// score is the sum of its group_top (1 or 2) largest c, only the `keep` best groups (ties: the lower group) can be chosen from; `top` rounds of arg-max of c
 // among them (ties: the lower index); the weights are the chosen s, over their sum when renormalize.
 constexpr int kMaxRouteGroups = 64;
 __global__ void __launch_bounds__(32) moe_route_grouped_kernel(const float *__restrict__ z, const float *__restrict__ correction,
                                                               int32_t *__restrict__ top_expert, float *__restrict__ top_weight, int outputs,
-                                                              int top, int groups, int keep, int score_fn, int renormalize) {
+                                                              int top, int groups, int keep, int group_top, int score_fn,
+                                                              int renormalize) {
     __shared__ float s_s[kMaxExperts], c_s[kMaxExperts], gbest[kMaxRouteGroups];
     __shared__ int gkept[kMaxRouteGroups];
     pdl_launch_dependents();
@@ -205,9 +206,13 @@ __global__ void __launch_bounds__(32) moe_route_grouped_kernel(const float *__re
     if (groups > 1) {
         const int per = outputs / groups;
         for (int g = lane; g < groups; g += 32) {
-            float b = -INFINITY;
-            for (int e = 0; e < per; ++e) b = fmaxf(b, c_s[g * per + e]);
-            gbest[g] = b;
+            float b = -INFINITY, second = -INFINITY;
+            for (int e = 0; e < per; ++e) {
+                const float v = c_s[g * per + e];
+                second = fmaxf(second, fminf(b, v));
+                b = fmaxf(b, v);
+            }
+            gbest[g] = group_top > 1 && per > 1 ? b + second : b;
             gkept[g] = 0;
         }
         __syncwarp();
@@ -466,13 +471,13 @@ bool hyb_moe_route(const void *h, const float *w_router, const float *w_row_gate
 }
 
 bool hyb_moe_route_grouped(const void *h, const float *w_router, const float *correction, int32_t *top_expert, float *top_weight, int64_t T,
-                           int64_t width, int64_t outputs, int64_t top, int64_t groups, int64_t keep, int32_t score_fn, int32_t renormalize,
-                           uint32_t dtype, cudaStream_t stream) {
+                           int64_t width, int64_t outputs, int64_t top, int64_t groups, int64_t keep, int32_t group_top, int32_t score_fn,
+                           int32_t renormalize, uint32_t dtype, cudaStream_t stream) {
     if (T <= 0) return true;
     if (!hybrid::known_dtype(dtype, "atoma_moe_route_grouped")) return false;
     if (groups <= 1) groups = 1, keep = 1;
     if (!h || !w_router || !top_expert || !top_weight || width <= 0 || outputs <= 0 || outputs > kMaxExperts || top <= 0 || top > outputs ||
-        groups > kMaxRouteGroups || outputs % groups || keep <= 0 || keep > groups || (score_fn != ATOMA_SCORE_SIGMOID && score_fn != ATOMA_SCORE_SOFTMAX)) {
+        groups > kMaxRouteGroups || outputs % groups || keep <= 0 || keep > groups || group_top < 0 || group_top > 2 || (score_fn != ATOMA_SCORE_SIGMOID && score_fn != ATOMA_SCORE_SOFTMAX)) {
         set_status(kErrInvalidArg, "atoma_moe_route_grouped: null argument, top %lld of %lld outputs (at most %d), or %lld of %lld groups (at most %d, equal sizes)",
                    static_cast<long long>(top), static_cast<long long>(outputs), kMaxExperts, static_cast<long long>(keep),
                    static_cast<long long>(groups), kMaxRouteGroups);
@@ -499,7 +504,7 @@ bool hyb_moe_route_grouped(const void *h, const float *w_router, const float *co
     if (!hybrid::launched(e, "moe_logits_kernel")) return false;
     return hybrid::launched(launch_ex(moe_route_grouped_kernel, dim3(static_cast<unsigned>(T)), dim3(32), 0, stream, static_cast<const float *>(z),
                                       correction, top_expert, top_weight, rows, static_cast<int>(top), static_cast<int>(groups),
-                                      static_cast<int>(keep), static_cast<int>(score_fn), static_cast<int>(renormalize)),
+                                      static_cast<int>(keep), static_cast<int>(group_top), static_cast<int>(score_fn), static_cast<int>(renormalize)),
                             "moe_route_grouped_kernel");
 }
 
@@ -617,9 +622,9 @@ extern "C" void atoma_moe_experts(const atoma_moe_args *args, const void **exper
     hyb_moe_experts(*args, expert_out, pair_row, static_cast<cudaStream_t>(stream));
 }
 extern "C" void atoma_moe_route_grouped(const void *h, const float *w_router, const float *correction, int32_t *top_expert, float *top_weight,
-                                        int64_t T, int64_t width, int64_t outputs, int64_t top, int64_t groups, int64_t keep, int32_t score_fn,
-                                        int32_t renormalize, uint32_t dtype, atoma_stream_t stream) {
+                                        int64_t T, int64_t width, int64_t outputs, int64_t top, int64_t groups, int64_t keep, int32_t group_top,
+                                        int32_t score_fn, int32_t renormalize, uint32_t dtype, atoma_stream_t stream) {
     clear_status();
-    hyb_moe_route_grouped(h, w_router, correction, top_expert, top_weight, T, width, outputs, top, groups, keep, score_fn, renormalize, dtype,
+    hyb_moe_route_grouped(h, w_router, correction, top_expert, top_weight, T, width, outputs, top, groups, keep, group_top, score_fn, renormalize, dtype,
                           static_cast<cudaStream_t>(stream));
 }

@@ -22,7 +22,7 @@ namespace atoma {
 
 extern int g_hybrid_debug;   // bit 1: general kernels only; bit 4: scans with many rows per lane
 bool hyb_head_project_ld(const void *, int64_t, int64_t, const void *, void *, int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, int32_t,
-                         uint32_t, cudaStream_t);   // latent_attention.cu
+                         uint32_t, cudaStream_t, const void * = nullptr, int64_t = 0);   // latent_attention.cu
 
 namespace {
 
@@ -98,12 +98,13 @@ __global__ void __launch_bounds__(256) tap_filter_kernel(const atoma_tap_filter_
     const int ctx = a.context_lens[b];
     const T *in = static_cast<const T *>(a.in);
     const float *hist = a.history ? a.history + static_cast<int64_t>(a.state_slots[b]) * a.history_stride : nullptr;
-    const float cur = to_f(in[t * a.ld_in + c]);
-    float f1 = 0.f, f2 = 0.f;
+    const float ib = a.in_bias ? a.in_bias[c] : 0.f;
+    const float cur = to_f(in[t * a.ld_in + c]) + ib;
+    float f1 = a.bias1 ? a.bias1[c] : 0.f, f2 = 0.f;
     for (int j = 0; j + 1 < taps; ++j) {
         const int back = taps - 1 - j;
         float v = 0.f;
-        if (i - back >= 0) v = to_f(in[(t - back) * a.ld_in + c]);
+        if (i - back >= 0) v = to_f(in[(t - back) * a.ld_in + c]) + ib;
         else if (ctx + i - back >= 0 && hist) v = hist[static_cast<int64_t>(taps - 1 + i - back) * C + c];
         f1 = fmaf(a.w1[c * taps + j], v, f1);
         if (a.w2) f2 = fmaf(a.w2[c * taps + j], v, f2);
@@ -148,13 +149,19 @@ __global__ void __launch_bounds__(128) tap_filter_vec_kernel(const atoma_tap_fil
             }
         }
     }
+    float ib[8], ob[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+        ib[e] = a.in_bias ? a.in_bias[c0 + e] : 0.f;
+        ob[e] = a.bias1 ? a.bias1[c0 + e] : 0.f;
+    }
     auto row8 = [&](int64_t t, float *v) {
         const uint4 r = *reinterpret_cast<const uint4 *>(in + t * a.ld_in + c0);
         const uint32_t u[4] = {r.x, r.y, r.z, r.w};
 #pragma unroll
         for (int e = 0; e < 4; ++e) {
-            v[2 * e] = __uint_as_float(u[e] << 16);
-            v[2 * e + 1] = __uint_as_float(u[e] & 0xffff0000u);
+            v[2 * e] = __uint_as_float(u[e] << 16) + ib[2 * e];
+            v[2 * e + 1] = __uint_as_float(u[e] & 0xffff0000u) + ib[2 * e + 1];
         }
     };
     float win[TAPS > 1 ? TAPS - 1 : 1][8];                     // win[k]: the input TAPS - 1 - k tokens back
@@ -182,7 +189,7 @@ __global__ void __launch_bounds__(128) tap_filter_vec_kernel(const atoma_tap_fil
         row8(t, cur);
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
-            float x = 0.f, y = 0.f;
+            float x = ob[e], y = 0.f;
 #pragma unroll
             for (int k = 0; k < TAPS - 1; ++k) {
                 x = fmaf(w1[e][k], win[k][e], x);
@@ -238,6 +245,7 @@ __global__ void __launch_bounds__(256) tap_history_kernel(const atoma_tap_filter
     if (n <= 0) return;
     float *hist = a.history + static_cast<int64_t>(a.state_slots[b]) * a.history_stride;
     const T *in = static_cast<const T *>(a.in);
+    const float ib = a.in_bias ? a.in_bias[c] : 0.f;
     float old[kMaxTaps];
 #pragma unroll
     for (int k = 0; k < kMaxTaps; ++k) old[k] = (k < keep && k + n < keep && ctx - keep + k + n >= 0) ? hist[static_cast<int64_t>(k + n) * C + c] : 0.f;
@@ -245,7 +253,7 @@ __global__ void __launch_bounds__(256) tap_history_kernel(const atoma_tap_filter
     for (int k = 0; k < kMaxTaps; ++k) {
         if (k >= keep) break;
         const int rel = n - keep + k;
-        hist[static_cast<int64_t>(k) * C + c] = rel >= 0 ? to_f(in[static_cast<int64_t>(q0 + rel) * a.ld_in + c]) : old[k];
+        hist[static_cast<int64_t>(k) * C + c] = rel >= 0 ? to_f(in[static_cast<int64_t>(q0 + rel) * a.ld_in + c]) + ib : old[k];
     }
 }
 
@@ -533,6 +541,17 @@ __global__ void __launch_bounds__(256) headnorm_gate_kernel(const float *__restr
 // ---------------------------------------------------------------------------------------------
 // rotary positions
 // ---------------------------------------------------------------------------------------------
+// sin and cos of pos * (freq + freq_lo), times amplitude.  The product is kept to twice float32's precision (its rounding error and the
+// part of the frequency that float32 drops turn the pair by a correction): at position 10^5 a plain float32 angle is off by 4e-3.
+__device__ __forceinline__ void turn(float pos, float freq, float freq_lo, float amplitude, float &sn, float &cs) {
+    const float ang = pos * freq;
+    const float rest = fmaf(pos, freq, -ang) + pos * freq_lo;
+    float s, c;
+    sincosf(ang, &s, &c);
+    sn = amplitude * fmaf(rest, c, s);
+    cs = amplitude * fmaf(-rest, s, c);
+}
+
 // buf [n] float32 (one warp's): the first 2 pairs entries turned by sign * pos * freq, written to dst as T.
 template <typename T>
 __device__ __forceinline__ void rotate_store(const float *buf, int n, const float *__restrict__ freq, int pairs, int interleaved, float pos,
@@ -567,19 +586,22 @@ __global__ void __launch_bounds__(256) qkv_headnorm_rope_cache_kernel(const atom
         const int hd = is_q ? u : (is_k ? u - H : u - H - G);
         if (!is_q && slot < 0) continue;
         const int n = (is_q || is_k) ? D : V;
-        const T *src = row + (is_q ? a.q_off + hd * D : (is_k ? a.k_off + hd * D : a.v_off + hd * V));
+        const int64_t col = is_q ? a.q_off + hd * D : (is_k ? a.k_off + hd * D : a.v_off + hd * V);
+        const T *src = row + col;
+        const float *bias = a.bias ? a.bias + col : nullptr;
         const float *w = is_q ? a.q_weight : (is_k ? a.k_weight : nullptr);
         float ss = 0.f;
         for (int c = lane; c < n; c += 32) {
-            const float v = to_f(src[c]);
+            const float v = to_f(src[c]) + (bias ? bias[c] : 0.f);
             buf[c] = v;
             ss = fmaf(v, v, ss);
         }
-        if (w) {
+        if (w || (a.unit_norm && (is_q || is_k))) {
 #pragma unroll
             for (int s = 16; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
-            const float inv = 1.0f / sqrtf(ss / static_cast<float>(n) + a.eps);
-            for (int c = lane; c < n; c += 32) buf[c] = buf[c] * inv * w[c];
+            float inv = 1.0f / sqrtf(ss / static_cast<float>(n) + a.eps);
+            if (is_q && a.q_head_scale) inv *= a.q_head_scale[hd];
+            for (int c = lane; c < n; c += 32) buf[c] = w ? buf[c] * inv * w[c] : buf[c] * inv;
         }
         __syncwarp();
         T *dst = is_q ? static_cast<T *>(a.q_out) + (t * H + hd) * D
@@ -616,7 +638,8 @@ __global__ void __launch_bounds__(256) rotate_heads_kernel(T *__restrict__ x, co
 template <typename T>
 __global__ void __launch_bounds__(kRowThreads) latent_norm_rope_cache_kernel(const T *__restrict__ proj, int64_t ld,
                                                                              const float *__restrict__ q_w, const float *__restrict__ kv_w,
-                                                                             const float *__restrict__ freq, int pairs, int interleaved,
+                                                                             const float *__restrict__ freq, const float *__restrict__ freq_lo,
+                                                                             float amplitude, int pairs, int interleaved,
                                                                              const int64_t *__restrict__ positions,
                                                                              const int64_t *__restrict__ slots, T *__restrict__ cq_out,
                                                                              T *__restrict__ cache, int q_rank, int kv_rank, int rot_dim,
@@ -650,7 +673,7 @@ __global__ void __launch_bounds__(kRowThreads) latent_norm_rope_cache_kernel(con
     for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
         const int ia = interleaved ? 2 * i : i, ib = interleaved ? 2 * i + 1 : i + pairs;
         float sn, cs;
-        sincosf(pos * freq[i], &sn, &cs);
+        turn(pos, freq[i], freq_lo ? freq_lo[i] : 0.f, amplitude, sn, cs);
         const float u = to_f(kr[ia]), v = to_f(kr[ib]);
         dst[kv_rank + ia] = from_f<T>(u * cs - v * sn);
         dst[kv_rank + ib] = from_f<T>(v * cs + u * sn);
@@ -660,8 +683,8 @@ __global__ void __launch_bounds__(kRowThreads) latent_norm_rope_cache_kernel(con
 
 // q_lat[t, h, kv_rank + c] = the rotated part of query head h, float32
 template <typename T>
-__global__ void __launch_bounds__(256) latent_query_rope_kernel(const T *__restrict__ q, const float *__restrict__ freq, int pairs,
-                                                                int interleaved, const int64_t *__restrict__ positions,
+__global__ void __launch_bounds__(256) latent_query_rope_kernel(const T *__restrict__ q, const float *__restrict__ freq,
+                                                                const float *__restrict__ freq_lo, float amplitude, int pairs, int interleaved, const int64_t *__restrict__ positions,
                                                                 float *__restrict__ q_lat, int H, int dim, int rot_dim, int kv_rank) {
     pdl_launch_dependents();
     pdl_wait();
@@ -673,7 +696,7 @@ __global__ void __launch_bounds__(256) latent_query_rope_kernel(const T *__restr
         const int ia = interleaved ? 2 * i : i, ib = interleaved ? 2 * i + 1 : i + pairs;
         const T *src = q + (t * H + h) * hs + dim;
         float sn, cs;
-        sincosf(pos * freq[i], &sn, &cs);
+        turn(pos, freq[i], freq_lo ? freq_lo[i] : 0.f, amplitude, sn, cs);
         const float u = to_f(src[ia]), v = to_f(src[ib]);
         float *dst = q_lat + (t * H + h) * row + kv_rank;
         dst[ia] = u * cs - v * sn;
@@ -828,7 +851,7 @@ bool hyb_qkv_headnorm_rope_cache(const atoma_qkv_rope_args &a, cudaStream_t stre
     if (!a.proj || !a.q_out || !a.positions || a.H <= 0 || a.G <= 0 || a.H % a.G || a.dim <= 0 || a.vdim <= 0 ||
         (a.slot_mapping && (!a.k_cache || !a.v_cache)) || a.q_off < 0 || a.k_off < 0 || a.v_off < 0 || a.q_off + a.H * a.dim > a.ld ||
         a.k_off + a.G * a.dim > a.ld || a.v_off + a.G * a.vdim > a.ld || a.rot_pairs < 0 || 2 * a.rot_pairs > a.dim || a.v_pairs < 0 ||
-        2 * a.v_pairs > a.vdim || (a.rot_pairs > 0 && !a.qk_freq)) {
+        2 * a.v_pairs > a.vdim || (a.rot_pairs > 0 && !a.qk_freq) || (a.q_head_scale && !a.q_weight && !a.unit_norm)) {
         set_status(kErrInvalidArg, "atoma_qkv_headnorm_rope_cache: null argument, columns outside the row, or more rotated entries than a head has");
         return false;
     }
@@ -857,7 +880,7 @@ bool hyb_rotate_heads(void *x, const int64_t *positions, const float *freq, int6
 #undef CALL
 }
 
-bool hyb_latent_norm_rope_cache(const void *proj, int64_t ld, const float *q_w, const float *kv_w, const float *freq, int64_t pairs,
+bool hyb_latent_norm_rope_cache(const void *proj, int64_t ld, const float *q_w, const float *kv_w, const float *freq, const float *freq_lo, float amplitude, int64_t pairs,
                                 int32_t interleaved, const int64_t *positions, const int64_t *slots, void *cq_out, void *cache, int64_t T,
                                 int64_t q_rank, int64_t kv_rank, int64_t rot_dim, float eps, uint32_t dtype, cudaStream_t stream) {
     if (T <= 0) return true;
@@ -868,14 +891,14 @@ bool hyb_latent_norm_rope_cache(const void *proj, int64_t ld, const float *q_w, 
         return false;
     }
 #define CALL(TT) launch_ex(latent_norm_rope_cache_kernel<TT>, dim3(static_cast<unsigned>(T)), dim3(kRowThreads), 0, stream, \
-                           static_cast<const TT *>(proj), ld, q_w, kv_w, freq, static_cast<int>(pairs), interleaved, positions, slots, \
+                           static_cast<const TT *>(proj), ld, q_w, kv_w, freq, freq_lo, amplitude, static_cast<int>(pairs), interleaved, positions, slots, \
                            static_cast<TT *>(cq_out), static_cast<TT *>(cache), static_cast<int>(q_rank), static_cast<int>(kv_rank), \
                            static_cast<int>(rot_dim), eps)
     return hybrid::launched(HYB_DISPATCH(dtype, CALL), "latent_norm_rope_cache_kernel");
 #undef CALL
 }
 
-bool hyb_latent_query_absorb_rope(const void *q, const void *w_uk, const float *freq, int64_t pairs, int32_t interleaved,
+bool hyb_latent_query_absorb_rope(const void *q, const void *w_uk, const float *freq, const float *freq_lo, float amplitude, int64_t pairs, int32_t interleaved,
                                   const int64_t *positions, float *q_lat, int64_t T, int64_t H, int64_t dim, int64_t rot_dim, int64_t kv_rank,
                                   uint32_t dtype, cudaStream_t stream) {
     if (T <= 0) return true;
@@ -888,21 +911,21 @@ bool hyb_latent_query_absorb_rope(const void *q, const void *w_uk, const float *
     const int64_t hs = dim + rot_dim, row = kv_rank + rot_dim;
     if (!hyb_head_project_ld(q, H * hs, hs, w_uk, q_lat, H * row, row, T, H, dim, kv_rank, 1, dtype, stream)) return false;
     if (rot_dim == 0) return true;
-#define CALL(TT) launch_ex(latent_query_rope_kernel<TT>, dim3(static_cast<unsigned>(T)), dim3(256), 0, stream, static_cast<const TT *>(q), freq, \
+#define CALL(TT) launch_ex(latent_query_rope_kernel<TT>, dim3(static_cast<unsigned>(T)), dim3(256), 0, stream, static_cast<const TT *>(q), freq, freq_lo, amplitude, \
                            static_cast<int>(pairs), interleaved, positions, q_lat, static_cast<int>(H), static_cast<int>(dim), \
                            static_cast<int>(rot_dim), static_cast<int>(kv_rank))
     return hybrid::launched(HYB_DISPATCH(dtype, CALL), "latent_query_rope_kernel");
 #undef CALL
 }
 
-bool hyb_latent_expand_values(const float *o_lat, const void *w_uv, void *out, int64_t T, int64_t H, int64_t vdim, int64_t kv_rank, int64_t row,
-                              uint32_t dtype, cudaStream_t stream) {
-    if (row < kv_rank) {
-        set_status(kErrInvalidArg, "atoma_latent_expand_values: rows of %lld entries for a latent of %lld", static_cast<long long>(row),
+bool hyb_latent_expand_values(const float *o_lat, const void *w_uv, const void *gate, int64_t ld_gate, void *out, int64_t T, int64_t H, int64_t vdim,
+                              int64_t kv_rank, int64_t row, uint32_t dtype, cudaStream_t stream) {
+    if (row < kv_rank || (gate && ld_gate < H * vdim)) {
+        set_status(kErrInvalidArg, "atoma_latent_expand_values: rows of %lld entries for a latent of %lld, or a gate row shorter than the heads", static_cast<long long>(row),
                    static_cast<long long>(kv_rank));
         return false;
     }
-    return hyb_head_project_ld(o_lat, H * row, row, w_uv, out, H * vdim, vdim, T, H, vdim, kv_rank, 0, dtype, stream);
+    return hyb_head_project_ld(o_lat, H * row, row, w_uv, out, H * vdim, vdim, T, H, vdim, kv_rank, 0, dtype, stream, gate, ld_gate);
 }
 
 }  // namespace atoma
@@ -957,25 +980,25 @@ extern "C" void atoma_rotate_heads(void *x, const int64_t *positions, const floa
     hyb_rotate_heads(x, positions, freq, T, H, n, pairs, interleaved, sign, dtype, static_cast<cudaStream_t>(stream));
 }
 
-extern "C" void atoma_latent_norm_rope_cache(const void *proj, int64_t ld, const float *q_weight, const float *kv_weight, const float *freq,
+extern "C" void atoma_latent_norm_rope_cache(const void *proj, int64_t ld, const float *q_weight, const float *kv_weight, const float *freq, const float *freq_lo, float amplitude,
                                              int64_t pairs, int32_t interleaved, const int64_t *positions, const int64_t *slot_mapping,
                                              void *cq_out, void *cache, int64_t T, int64_t q_rank, int64_t kv_rank, int64_t rot_dim, float eps,
                                              uint32_t dtype, atoma_stream_t stream) {
     clear_status();
-    hyb_latent_norm_rope_cache(proj, ld, q_weight, kv_weight, freq, pairs, interleaved, positions, slot_mapping, cq_out, cache, T, q_rank, kv_rank,
+    hyb_latent_norm_rope_cache(proj, ld, q_weight, kv_weight, freq, freq_lo, amplitude, pairs, interleaved, positions, slot_mapping, cq_out, cache, T, q_rank, kv_rank,
                                rot_dim, eps, dtype, static_cast<cudaStream_t>(stream));
 }
 
-extern "C" void atoma_latent_query_absorb_rope(const void *q, const void *w_uk, const float *freq, int64_t pairs, int32_t interleaved,
+extern "C" void atoma_latent_query_absorb_rope(const void *q, const void *w_uk, const float *freq, const float *freq_lo, float amplitude, int64_t pairs, int32_t interleaved,
                                                const int64_t *positions, float *q_lat, int64_t T, int64_t H, int64_t dim, int64_t rot_dim,
                                                int64_t kv_rank, uint32_t dtype, atoma_stream_t stream) {
     clear_status();
-    hyb_latent_query_absorb_rope(q, w_uk, freq, pairs, interleaved, positions, q_lat, T, H, dim, rot_dim, kv_rank, dtype,
+    hyb_latent_query_absorb_rope(q, w_uk, freq, freq_lo, amplitude, pairs, interleaved, positions, q_lat, T, H, dim, rot_dim, kv_rank, dtype,
                                  static_cast<cudaStream_t>(stream));
 }
 
-extern "C" void atoma_latent_expand_values(const float *o_lat, const void *w_uv, void *out, int64_t T, int64_t H, int64_t vdim, int64_t kv_rank,
-                                           int64_t row, uint32_t dtype, atoma_stream_t stream) {
+extern "C" void atoma_latent_expand_values(const float *o_lat, const void *w_uv, const void *gate, int64_t ld_gate, void *out, int64_t T, int64_t H,
+                                           int64_t vdim, int64_t kv_rank, int64_t row, uint32_t dtype, atoma_stream_t stream) {
     clear_status();
-    hyb_latent_expand_values(o_lat, w_uv, out, T, H, vdim, kv_rank, row, dtype, static_cast<cudaStream_t>(stream));
+    hyb_latent_expand_values(o_lat, w_uv, gate, ld_gate, out, T, H, vdim, kv_rank, row, dtype, static_cast<cudaStream_t>(stream));
 }

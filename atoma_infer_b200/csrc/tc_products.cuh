@@ -4,7 +4,7 @@
 // A is read as float32 or bfloat16 (converted while it is staged), B is bfloat16 with arbitrary element strides (so a
 // weight stored [k][n] needs no transposed copy), O is float32 or bfloat16.  In grouped mode the row tiles belong to
 // experts (tile_expert) and B(z) is the tile's expert; with GLU the tile computes the gate and the up product of the same
-// rows and stores the clamped gated activation.
+// rows and stores the clamped gated activation; the gates of a linear recurrent unit are two products of the same rows as well.
 // 64 x 64 x 32 tiles, four warps of 32 x 32.  bfloat16 operands with contiguous, 16-byte aligned k runs (the experts' case) go
 // through a three-stage cp.async ring, so that a CTA keeps two tiles of weights in flight while it multiplies a third — at
 // decode sizes the product is a pure weight stream; otherwise the next tile's operands are fetched into registers
@@ -31,7 +31,15 @@ struct GemmArgs {
     const int32_t *tile_expert, *meta, *row_pair;
     const float *out_weight;   // per pair, applied to the output row (nullptr: none)
     float limit, alpha, shift; // GLU epilogue
+    const __nv_bfloat16 *gate; // plain epilogue: the result times sigmoid(gate[m, z o_zs + n]), row stride ld_gate (nullptr: none)
+    int64_t ld_gate;
+    // kEpiLru epilogue: the gates of a real-gated linear recurrent unit (gated_lru.cu); channel z N + n
+    const float *bias_r, *bias_i, *rate;
+    float *decay, *input;
+    int64_t ld_state;
 };
+
+enum Epilogue { kEpiPlain = 0, kEpiGlu = 1, kEpiLru = 2 };   // kEpiGlu, kEpiLru: two products of the same rows (B's next N rows)
 
 constexpr int kTM = 64, kTN = 64, kTK = 32, kLd = kTK + 8, kStages = 3;
 
@@ -65,8 +73,16 @@ __device__ __forceinline__ uint4 fetch8(const TS *p, int64_t stride, int nvalid,
     return pack8(v);
 }
 
-template <typename TA, typename TO, bool GLU>
+// decay = exp(log a) and input = sqrt(1 - a^2) i u with log a = rate * sigmoid(r), i = sigmoid(ipre); 1 - a^2 = -expm1(2 log a).
+__device__ __forceinline__ void lru_gates(float rpre, float ipre, float rate, float u, float &decay, float &input) {
+    const float log_a = rate * hybrid::sigmoidf_(rpre);
+    decay = expf(log_a);
+    input = sqrtf(-expm1f(2.f * log_a)) * hybrid::sigmoidf_(ipre) * u;
+}
+
+template <typename TA, typename TO, int EPI>
 __global__ void __launch_bounds__(128) gemm_kernel(const GemmArgs p) {
+    constexpr bool GLU = EPI != kEpiPlain;
     __shared__ __align__(16) __nv_bfloat16 As[kStages][kTM][kLd], Bs[kStages][kTN][kLd], Us[GLU ? kStages : 1][GLU ? kTN : 1][kLd];
     pdl_launch_dependents();
     pdl_wait();
@@ -208,8 +224,19 @@ __global__ void __launch_bounds__(128) gemm_kernel(const GemmArgs p) {
                     const int n = n0 + wn * 32 + ni * 8 + 2 * t4 + e;
                     if (n >= p.N) continue;
                     float v = acc[mi][ni][half * 2 + e];
-                    if constexpr (GLU) v = hybrid::glu_clamped(v, acu[mi][ni][half * 2 + e], p.limit, p.alpha, p.shift);
-                    else v *= ow;
+                    if constexpr (EPI == kEpiLru) {
+                        const int64_t c = z * p.N + n;
+                        float d, in;
+                        lru_gates(v + p.bias_r[c], acu[mi][ni][half * 2 + e] + p.bias_i[c], p.rate[c], hybrid::to_f(A[static_cast<int64_t>(m) * p.lda + n]), d, in);
+                        p.decay[static_cast<int64_t>(m) * p.ld_state + c] = d;
+                        p.input[static_cast<int64_t>(m) * p.ld_state + c] = in;
+                        continue;
+                    }
+                    if constexpr (EPI == kEpiGlu) v = hybrid::glu_clamped(v, acu[mi][ni][half * 2 + e], p.limit, p.alpha, p.shift);
+                    else {
+                        v *= ow;
+                        if (p.gate) v *= hybrid::sigmoidf_(hybrid::to_f(p.gate[static_cast<int64_t>(m) * p.ld_gate + z * p.o_zs + n]));
+                    }
                     O[static_cast<int64_t>(m) * p.ldo + n] = hybrid::from_f<TO>(v);
                 }
         }

@@ -1,8 +1,7 @@
 """Hybrid (attention + recurrent) decoder models: description, device layout and the step executor's host side.
 
-A model family (atoma_infer_b200/lilovik.py is the first, patadra.py the second, nemasun.py the third) describes
-itself as a `HybridSpec` — a list of layer RUNS, each a mixer (sigmoid attention, minGRU, latent attention or softmax
-attention) with its sizes and constants and an optional feed-forward (gated dense, or a mixture of experts) — and hands over its
+A model family (atoma_infer_b200/lilovik.py, patadra.py, nemasun.py, surinex.py, mobunex.py) describes itself as a
+`HybridSpec` — a list of layer RUNS, each a mixer (attention of some kind, a recurrence, or a pair of them) with its sizes and constants and an optional feed-forward (gated dense, or a mixture of experts) — and hands over its
 weights under the generic names below.  A design that runs a span of layers several times lists every run;
 runs that name the same `source` share one copy of the weights and have caches of their own.  `HybridExecutor` lays them out
 on the device, owns the paged key/value caches and the recurrent-state slots, and runs one step of a MIXED
@@ -39,6 +38,13 @@ Parallel blocks (block_style "parallel": one norm per layer, x += mixer(f1(h)) +
                         [channels, taps'], r_a_log, r_dt_bias [H'], r_head_norm [vdim'], r_w_o [width, H' vdim']
                   out_norm_a, out_norm_b [width]
   the model: pass_vectors [passes, width] float32 (the vector added at the start of every pass over a looped span)
+Post-norm blocks (block_style "postnorm": x <- norm1(alpha x + mixer(x)), x <- norm2(alpha x + ff(x)), then an average over depth):
+  norm1, norm2 [width]   depth_w [layer index + 2] float32 (embedding output, results of the layers so far)   the model: embed_norm [width]
+  softmax attention: w_q, w_k, w_v and their biases b_q, b_k, b_v, head_scale [H] (factor of a head's scores), w_o
+  latent attention as for parallel blocks, with w_g [H vdim, width] (output gate)
+  linear recurrent unit: w_y, w_x [S, width], b_y, b_x [S], tap_w [S, taps], tap_b [S], gate_r, gate_i [blocks, n, n] stored [out, in], gate_r_b,
+                         gate_i_b [S], rate [S] (log of the decay at an open gate, <= 0), w_o [width, S]
+  dense: w_gate_up [2 ff, width], w_down [width, ff]     experts: as for blocks on residual lanes
 The executor stacks the projections that read the same input into one matrix (rows padded to a multiple of 8).
 """
 from __future__ import annotations
@@ -57,10 +63,10 @@ from .ops import AtomaError
 from .scheduler import StepPlan
 from .worker import InputStager, SequenceInput
 
-MIXER_ATTENTION, MIXER_MINGRU, MIXER_LATENT, MIXER_SOFTMAX, MIXER_GLA, MIXER_PAIR = 0, 1, 2, 3, 4, 5
+MIXER_ATTENTION, MIXER_MINGRU, MIXER_LATENT, MIXER_SOFTMAX, MIXER_GLA, MIXER_PAIR, MIXER_LRU = 0, 1, 2, 3, 4, 5, 6
 LONG_PORTION = 128        # tokens of a sequence in one step from which attention runs on the tensor-memory prefill kernel
                           # (latent attention: on expanded keys and values; softmax attention: on gathered ones)
-BLOCK_STYLES = {"sandwich": 0, "prenorm": 1, "lanes": 2, "parallel": 3}
+BLOCK_STYLES = {"sandwich": 0, "prenorm": 1, "lanes": 2, "parallel": 3, "postnorm": 4}
 SCORE_FNS = {"sigmoid": 0, "softmax": 1}
 ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2}
 DTYPE_CODES = {torch.bfloat16: 1, torch.float32: 2}
@@ -101,8 +107,9 @@ class LatentAttentionSpec:
     scale: float
     window: int = 0                # 0 = every earlier token is visible
     sink: bool = False             # a learned per-head term of the softmax denominator
-    rot_dim: int = 0               # parallel blocks: rotated entries per query head and of the one key part all heads share
+    rot_dim: int = 0               # parallel, post-norm blocks: rotated entries per query head and of the one key part all heads share
     rotary: Optional["RotarySpec"] = None
+    out_gate: bool = False         # post-norm blocks: heads' outputs times sigmoid(W h) before the output projection
 
 
 @dataclass(frozen=True)
@@ -119,17 +126,34 @@ class SoftmaxAttentionSpec:
     values_are_keys: bool = False  # no value projection: the values are the key projections before their norm
     out_gate: bool = False         # heads' outputs times sigmoid(W h) before the output projection
     distance_bias: bool = False    # weights carry dist_bias [rows, heads]
+    bias: bool = False             # post-norm blocks: the projections have biases
+    head_scale: bool = False       # post-norm blocks: a factor per head on the scores
 
 
 @dataclass(frozen=True)
 class RotarySpec:
     """Rotary positions on the first `dims` entries of a head: pair i turns by position * base^(-2 i / dims).  `scaling`
     (factor, low, high, original) stretches long wavelengths: a wavelength below original / high keeps its frequency, one
-    above original / low has it divided by factor, and in between the two are blended linearly in original / wavelength."""
+    above original / low has it divided by factor, and in between the two are blended linearly in original / wavelength.
+    `yarn` (factor, original, fast, slow) is the other stretching rule: pairs that turn more than `fast` times over the original length
+    keep their frequency, pairs that turn less than `slow` times have it divided by factor, in between the two are blended linearly in
+    the pair's index (its bounds rounded outwards to whole indices); cos and sin are multiplied by 0.1 ln(factor) + 1."""
     dims: int
     base: float = 10000.0
     interleaved: bool = False                 # pairs (2i, 2i + 1) instead of (i, i + dims / 2)
     scaling: Optional[Seq_[float]] = None     # (factor, low, high, original)
+    yarn: Optional[Seq_[float]] = None        # (factor, original, fast, slow)
+
+    @property
+    def amplitude(self) -> float:
+        return 1.0 if self.yarn is None else 0.1 * math.log(float(self.yarn[0])) + 1.0
+
+    def _yarn_share(self, i: int) -> float:
+        """How much of pair i's frequency is the divided one."""
+        _, original, fast, slow = (float(v) for v in self.yarn)
+        at = [self.dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(float(self.base))) for turns in (fast, slow)]
+        lo, hi = max(math.floor(at[0]), 0), min(math.ceil(at[1]), self.dims - 1)
+        return min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
 
     def frequencies(self) -> List[float]:
         out = []
@@ -143,6 +167,9 @@ class RotarySpec:
                 elif wave >= original / high:
                     t = (original / wave - low) / (high - low)
                     f = (1.0 - t) * f / factor + t * f
+            if self.yarn is not None:
+                share = self._yarn_share(i)
+                f = f / float(self.yarn[0]) * share + f * (1.0 - share)
             out.append(f)
         return out
 
@@ -191,6 +218,17 @@ class MixerPairSpec:
 
 
 @dataclass(frozen=True)
+class LinearRecurrentSpec:
+    """Recurrent block with a real-gated linear recurrent unit: two branches of `width`, one through an activation, the other through a
+    short causal filter and S <- a S + sqrt(1 - a^2) i u with a per-channel, per-token decay a and input gate i from block-diagonal
+    matrices; the state times the activated branch is projected out."""
+    width: int
+    blocks: int
+    taps: int = 4
+    act: str = "gelu_tanh"         # of the gate branch
+
+
+@dataclass(frozen=True)
 class ClampedMlpSpec:
     """Dense feed-forward W_down (g sigmoid(alpha g) (u + up_shift)) on g = min(W_gate h + b, limit), u = clamp(W_up h + b)."""
     ff: int
@@ -219,6 +257,7 @@ class MoeSpec:
     correction: bool = False       # a per-output term added to the scores for the choice only
     groups: int = 1                # router outputs form this many equal groups of neighbours ...
     keep_groups: int = 1           # ... of which only the best may be chosen from
+    group_top: int = 1             # a group is ranked by the sum of this many of its largest choice scores (1 or 2)
     identity: int = 0              # router outputs after the experts that hand the token's input through
     scale_input: bool = True       # the router's weight multiplies the expert's input (False: its output)
 
@@ -241,6 +280,7 @@ class LayerSpec:
     taps: int = 0                            # parallel blocks: taps of the filters on the sublayers' inputs (0: none)
     add_embedding: bool = False              # parallel blocks: the embedding rows are added to the stream before the layer
     pass_vector: Optional[int] = None        # ... and this row of weights["pass_vectors"]
+    lru: Optional["LinearRecurrentSpec"] = None
 
 
 @dataclass(frozen=True)
@@ -260,10 +300,12 @@ class HybridSpec:
     side_dim: int = 0                        # width of one layer's part of the token side table
     lanes: int = 0                           # block_style "lanes": copies of the residual stream
     embed_scale: float = 1.0                 # block_style "lanes": the embedding row times this (no position signal)
+    residual_alpha: float = 1.0              # block_style "postnorm": the stream's factor in every sum
+    depth_average: bool = False              # block_style "postnorm": a layer hands on a weighted sum of every result so far
 
     @property
     def has_state(self) -> bool:
-        return any(l.mixer == "mingru" or l.taps > 1 or l.gla is not None or l.pair is not None for l in self.layers)
+        return any(l.mixer == "mingru" or l.taps > 1 or l.gla is not None or l.pair is not None or l.lru is not None for l in self.layers)
 
     def cache_bytes_per_token(self, dtype: torch.dtype) -> int:
         es = torch.empty((), dtype=dtype).element_size()
@@ -313,7 +355,7 @@ class HybridExecutor:
         if spec.block_style == "lanes":
             if not 1 <= spec.lanes <= 16:
                 raise AtomaError(f"{spec.lanes} residual lanes (1 to 16 are supported)")
-        elif spec.block_style == "parallel":
+        elif spec.block_style in ("parallel", "postnorm"):
             pass                  # positions enter through the mixers' rotations
         elif spec.position == "learned":
             self.pos_table = big(weights["pos"])
@@ -351,13 +393,14 @@ class HybridExecutor:
                 self.states.append(None)
                 self.latent_caches.append(None)
                 continue
-            if spec.block_style == "parallel":
-                if src in placed:
+            if spec.block_style in ("parallel", "postnorm"):
+                if src in placed and spec.block_style == "parallel":
                     C.memmove(C.byref(L), C.byref(placed[src]), C.sizeof(HybridLayer))     # same weights; caches, state and pass start below
                 else:
-                    self._place_parallel(L, i, ls, w, big, small)
+                    place = self._place_parallel if spec.block_style == "parallel" else self._place_postnorm
+                    place(L, i, ls, w, big, small)
                     placed[src] = L
-                self._parallel_run_state(L, i, ls, weights, small, rows)
+                self._run_state(L, i, ls, weights, small, rows)
                 continue
             if spec.block_style == "prenorm":
                 if src in placed:
@@ -422,6 +465,11 @@ class HybridExecutor:
         if self.side_table is not None:
             m.side_table, m.side_dim, m.side_table_width = self.side_table.data_ptr(), spec.side_dim, self.side_table.shape[1]
         m.lanes, m.embed_scale = spec.lanes, spec.embed_scale
+        if spec.block_style == "postnorm":
+            self.embed_norm = small(weights["embed_norm"])
+            if tuple(self.embed_norm.shape) != (spec.width,) or tuple(self.final_norm.shape) != (spec.width,):
+                raise AtomaError(f"norms of the embedding and the output have shapes {tuple(self.embed_norm.shape)}, {tuple(self.final_norm.shape)}")
+            m.embed_norm, m.residual_alpha = self.embed_norm.data_ptr(), spec.residual_alpha
         self._model = m
         self._stager = InputStager(device=dev, block_size=self.block_size, enable_chunked_prefill=True)
         self._extra_host = None
@@ -517,17 +565,21 @@ class HybridExecutor:
             if f.bias:
                 L.b_gate_up, L.b_down = small(w["b_gate_up"]).data_ptr(), small(w["b_down"]).data_ptr()
             return
-        e = ls.moe
+        self._place_routed(L, i, ls.moe, w, big, small)
+
+    @staticmethod
+    def _place_routed(L, i: int, e: MoeSpec, w: dict, big, small) -> None:
+        """Device copies and sizes of a mixture of experts whose router corrects and restricts its choice."""
         outputs = e.experts + e.identity
         if e.score not in SCORE_FNS:
             raise AtomaError(f"layer {i}: unknown router score {e.score!r}")
         if not 0 < e.top <= outputs or e.experts < 1:
             raise AtomaError(f"layer {i}: top {e.top} of {outputs} router outputs ({e.experts} experts)")
-        if e.groups < 1 or outputs % e.groups or not 1 <= e.keep_groups <= e.groups:
-            raise AtomaError(f"layer {i}: {outputs} router outputs in {e.groups} groups, {e.keep_groups} kept")
+        if e.groups < 1 or outputs % e.groups or not 1 <= e.keep_groups <= e.groups or e.group_top not in (1, 2):
+            raise AtomaError(f"layer {i}: {outputs} router outputs in {e.groups} groups, {e.keep_groups} kept, ranked by {e.group_top} scores")
         L.ff_kind, L.renormalize, L.score_fn, L.scale_input = 1, int(e.renormalize), SCORE_FNS[e.score], int(e.scale_input)
         L.experts, L.top, L.expert_ff, L.ff = e.experts, e.top, e.ff, e.shared_ff
-        L.identity_experts, L.route_groups, L.route_keep = e.identity, e.groups, e.keep_groups
+        L.identity_experts, L.route_groups, L.route_keep, L.route_group_top = e.identity, e.groups, e.keep_groups, e.group_top
         L.expert_limit, L.shared_limit, L.act_alpha, L.act_up_shift = e.limit, e.shared_limit, e.alpha, e.up_shift
         L.w_router = small(w["w_router"]).data_ptr()
         if e.correction:
@@ -536,17 +588,121 @@ class HybridExecutor:
         if e.shared_ff > 0:
             L.w_ff_in, L.w_down = big(w["w_ff_in"]).data_ptr(), big(w["w_down"]).data_ptr()
 
-    def _place_parallel(self, L, i: int, ls: LayerSpec, w: dict, big, small) -> None:
-        """Device copies and sizes of one parallel layer: the projections that read the mixer's input stacked into one matrix
-        (every part starts at a multiple of 8 rows, so that each has 16-byte aligned columns in the product)."""
-        W = self.spec.width
-
+    @staticmethod
+    def _shaped(i: int, w: dict):
+        """Lookup of a layer's tensor by its generic name, with the shape the description needs."""
         def need(name, shape):
             t = w.get(name)
             if t is None or tuple(t.shape) != tuple(shape):
                 raise AtomaError(f"layer {i}: tensor {name} is {None if t is None else tuple(t.shape)}, the description needs {tuple(shape)}")
             return t
+        return need
 
+    def _place_rotation(self, L, i: int, r: "RotarySpec", limit: int, small) -> None:
+        if r.dims > limit or r.dims % 2:
+            raise AtomaError(f"layer {i}: {r.dims} rotated entries in a part of {limit}")
+        f = torch.tensor(r.frequencies(), dtype=torch.float64)
+        hi = f.to(torch.float32)
+        L.qk_freq, L.qk_freq_lo = small(hi).data_ptr(), small(f - hi.double()).data_ptr()
+        L.rot_pairs, L.rot_interleaved, L.rot_amplitude = r.dims // 2, int(r.interleaved), r.amplitude
+
+    def _place_postnorm(self, L, i: int, ls: LayerSpec, w: dict, big, small) -> None:
+        """Device copies and sizes of one post-norm layer: the projections that read the stream stacked into one matrix (the parts start at
+        multiples of 8 rows, except that a latent layer's [c_q | c | rotated key part] are neighbours), their biases beside it."""
+        W = self.spec.width
+        need = self._shaped(i, w)
+        parts: List[torch.Tensor] = []
+        biases: List[torch.Tensor] = []
+
+        def stack(rows_of, bias=None) -> int:
+            at, n = sum(p.shape[0] for p in parts), sum(t.shape[0] for t in rows_of)
+            parts.extend(rows_of)
+            biases.append(bias.float() if bias is not None else torch.zeros(n))
+            pad = -n % 8
+            if pad:
+                parts.append(torch.zeros((pad, W), dtype=rows_of[0].dtype))
+                biases.append(torch.zeros(pad))
+            return at
+
+        L.norm1 = small(need("norm1", (W,))).data_ptr()
+        if self.spec.depth_average:
+            L.depth_w = small(need("depth_w", (i + 2,))).data_ptr()
+        if ls.mixer == "softmax_attention":
+            a = ls.softmax
+            if a.heads % a.kv_heads:
+                raise AtomaError(f"layer {i}: {a.kv_heads} kv heads do not divide {a.heads} heads")
+            if a.keep_first or a.values_are_keys or a.out_gate or a.distance_bias:
+                raise AtomaError(f"layer {i}: kept first tokens, values that are keys, output gates and distance tables are served on residual lanes")
+            L.mixer = MIXER_SOFTMAX
+            L.heads, L.kv_heads, L.dim, L.vdim, L.scale, L.window = a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window
+            bias = lambda name, n: need(name, (n,)) if a.bias else None
+            L.q_off = stack([need("w_q", (a.heads * a.dim, W))], bias("b_q", a.heads * a.dim))
+            L.k_off = stack([need("w_k", (a.kv_heads * a.dim, W))], bias("b_k", a.kv_heads * a.dim))
+            L.v_off = stack([need("w_v", (a.kv_heads * a.vdim, W))], bias("b_v", a.kv_heads * a.vdim))
+            if a.head_scale:
+                L.q_head_scale = small(need("head_scale", (a.heads,))).data_ptr()
+            L.w_o = big(need("w_o", (W, a.heads * a.vdim))).data_ptr()
+        elif ls.mixer == "latent_attention":
+            a = ls.latent
+            if a.sink:
+                raise AtomaError(f"layer {i}: post-norm blocks have no softmax sinks")
+            L.mixer = MIXER_LATENT
+            L.heads, L.kv_heads, L.dim, L.vdim = a.heads, 1, a.dim, a.vdim
+            L.q_rank, L.kv_rank, L.window, L.scale, L.rot_dim = a.q_rank, a.kv_rank, a.window, a.scale, a.rot_dim
+            stack([need("w_dq", (a.q_rank, W)), need("w_dkv", (a.kv_rank + a.rot_dim, W))])
+            if a.out_gate:
+                L.out_gate, L.g_off = 1, stack([need("w_g", (a.heads * a.vdim, W))])
+            L.dq_norm, L.dkv_norm = small(need("dq_norm", (a.q_rank,))).data_ptr(), small(need("dkv_norm", (a.kv_rank,))).data_ptr()
+            L.w_uq = big(need("w_uq", (a.heads * (a.dim + a.rot_dim), a.q_rank))).data_ptr()
+            L.w_uk = big(need("w_uk", (a.heads * a.dim, a.kv_rank))).data_ptr()
+            L.w_uv = big(need("w_uv", (a.heads * a.vdim, a.kv_rank))).data_ptr()
+            L.w_o = big(need("w_o", (W, a.heads * a.vdim))).data_ptr()
+            L.rot_amplitude = 1.0
+            if a.rot_dim > 0:
+                self._place_rotation(L, i, a.rotary or RotarySpec(dims=a.rot_dim), a.rot_dim, small)
+        elif ls.mixer == "lru":
+            d = ls.lru
+            if d.blocks < 1 or d.width % d.blocks:
+                raise AtomaError(f"layer {i}: {d.width} channels in {d.blocks} blocks")
+            if not 1 <= d.taps <= 16:
+                raise AtomaError(f"layer {i}: {d.taps} taps of the short filter (1 to 16 are supported)")
+            if d.act not in ACTIVATIONS:
+                raise AtomaError(f"layer {i}: unknown activation {d.act!r}")
+            n = d.width // d.blocks
+            L.mixer = MIXER_LRU
+            L.lru_width, L.lru_blocks, L.r_taps, L.act = d.width, d.blocks, d.taps, ACTIVATIONS[d.act]
+            L.q_off = stack([need("w_y", (d.width, W))], need("b_y", (d.width,)))
+            L.k_off = stack([need("w_x", (d.width, W))], need("b_x", (d.width,)))
+            L.r_tap_w, L.r_tap_bias = small(need("tap_w", (d.width, d.taps))).data_ptr(), small(need("tap_b", (d.width,))).data_ptr()
+            L.lru_w = big(torch.cat([need("gate_r", (d.blocks, n, n)), need("gate_i", (d.blocks, n, n))], 1)).data_ptr()
+            L.lru_bias_r, L.lru_bias_i = small(need("gate_r_b", (d.width,))).data_ptr(), small(need("gate_i_b", (d.width,))).data_ptr()
+            L.lru_rate = small(need("rate", (d.width,))).data_ptr()
+            L.w_o = big(need("w_o", (W, d.width))).data_ptr()
+        else:
+            raise AtomaError(f"layer {i}: post-norm blocks take the mixers softmax_attention, latent_attention and lru, not {ls.mixer!r}")
+        L.w_qkv, L.b_qkv = big(torch.cat(parts, 0)).data_ptr(), small(torch.cat(biases, 0)).data_ptr()
+        L.proj_cols = sum(p.shape[0] for p in parts)
+        L.has_mlp = 1 if ls.mlp is not None or ls.moe is not None else 0
+        if not L.has_mlp:
+            return
+        L.norm2 = small(need("norm2", (W,))).data_ptr()
+        if ls.mlp is not None:
+            if ls.mlp.act != "silu":
+                raise AtomaError(f"layer {i}: post-norm blocks have silu-gated feed-forwards, not {ls.mlp.act!r}")
+            L.ff_kind, L.ff = 0, ls.mlp.ff
+            L.w_gate_up, L.w_down = big(need("w_gate_up", (2 * L.ff, W))).data_ptr(), big(need("w_down", (W, L.ff))).data_ptr()
+            return
+        e = ls.moe
+        if e.identity or e.shared_limit or e.shared_gate:
+            raise AtomaError(f"layer {i}: identity experts and clamped or gated shared experts are served by other block styles")
+        self._place_routed(L, i, e, w, big, small)
+
+    def _place_parallel(self, L, i: int, ls: LayerSpec, w: dict, big, small) -> None:
+        """Device copies and sizes of one parallel layer: the projections that read the mixer's input stacked into one matrix
+        (every part starts at a multiple of 8 rows, so that each has 16-byte aligned columns in the product)."""
+        W = self.spec.width
+
+        need = self._shaped(i, w)
         parts: List[torch.Tensor] = []
         offsets: Dict[str, int] = {}
 
@@ -661,24 +817,26 @@ class HybridExecutor:
         L.w_qkv = big(torch.cat(parts, 0)).data_ptr()
 
     def state_floats(self, ls: LayerSpec) -> int:
-        """float32 entries of one sequence's state in one run of a parallel layer: [input history | mixer state]."""
+        """float32 entries of one sequence's state in one run of a parallel or post-norm layer: [input history | mixer state]."""
         n = max(0, ls.taps - 1) * self.spec.width
         if ls.gla is not None:
             n += ls.gla.heads * ls.gla.dim * ls.gla.vdim
         if ls.pair is not None:
             d = ls.pair.right
             n += max(0, d.taps - 1) * (2 * d.kv_heads * d.dim + d.heads * d.vdim) + d.heads * d.dim * d.vdim
+        if ls.lru is not None:
+            n += max(0, ls.lru.taps - 1) * ls.lru.width + ls.lru.width
         return n
 
-    def _parallel_run_state(self, L, i: int, ls: LayerSpec, weights: dict, small, rows: int) -> None:
-        """What one RUN of a parallel layer owns: its caches, its state rows, and what precedes it in the stream."""
+    def _run_state(self, L, i: int, ls: LayerSpec, weights: dict, small, rows: int) -> None:
+        """What one RUN of a parallel or post-norm layer owns: its caches, its state rows, and what precedes it in the stream."""
         dev, dtype = self.device, self.dtype
         kc = vc = lc = st = None
         if ls.mixer == "latent_attention":
             lc = torch.zeros((rows, ls.latent.kv_rank + ls.latent.rot_dim), dtype=dtype, device=dev)
             L.latent_cache = lc.data_ptr()
-        elif ls.mixer == "pair":
-            a = ls.pair.left
+        elif ls.mixer in ("pair", "softmax_attention"):
+            a = ls.pair.left if ls.pair is not None else ls.softmax
             kc = torch.zeros((rows, a.kv_heads, a.dim), dtype=dtype, device=dev)
             vc = torch.zeros((rows, a.kv_heads, a.vdim), dtype=dtype, device=dev)
             L.k_cache, L.v_cache = kc.data_ptr(), vc.data_ptr()
@@ -770,7 +928,7 @@ class HybridExecutor:
         hb.num_tokens, hb.num_seqs, hb.num_selected, hb.max_blocks = T, B, S, bt.shape[1]
         hb.max_query_len = max(c.count for c in chunks)
         hb.max_seq_len = max(c.start + c.count for c in chunks)
-        if self.spec.block_style in ("prenorm", "lanes"):
+        if self.spec.block_style in ("prenorm", "lanes", "postnorm"):
             long_ = [c for c in chunks if c.count >= LONG_PORTION]
             hb.long_seqs, hb.long_min_q = len(long_), LONG_PORTION
             hb.long_tokens, hb.long_ctx_sum = sum(c.count for c in long_), sum(c.start for c in long_)

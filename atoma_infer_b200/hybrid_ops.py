@@ -385,11 +385,11 @@ def softmax_attention_paged(q, k_cache, v_cache, positions, token_seq, block_tab
     return out
 
 
-def moe_route_grouped(h, w_router, correction, top, groups=1, keep=1, score="softmax", renormalize=True):
+def moe_route_grouped(h, w_router, correction, top, groups=1, keep=1, score="softmax", renormalize=True, group_top=1):
     T, E = h.shape[0], w_router.shape[0]
     idx = torch.empty((T, top), dtype=torch.int32, device=h.device)
     wgt = torch.empty((T, top), dtype=torch.float32, device=h.device)
-    _lib.lib().atoma_moe_route_grouped(_p(h), _p(w_router), _p(correction), _p(idx), _p(wgt), T, h.shape[1], E, top, groups, keep,
+    _lib.lib().atoma_moe_route_grouped(_p(h), _p(w_router), _p(correction), _p(idx), _p(wgt), T, h.shape[1], E, top, groups, keep, group_top,
                                        1 if score == "softmax" else 0, 1 if renormalize else 0, _CODES[h.dtype], _s())
     _check()
     return idx, wgt
@@ -452,7 +452,8 @@ def parallel_residual_norm(x, dtype, y_a=None, y_b=None, y_ff=None, norm_a=None,
     return h, trace
 
 
-def tap_filter(x, w1, w2, history, state_slots, token_seq, query_start, context_lens, residual: bool, act: int = 0):
+def tap_filter(x, w1, w2, history, state_slots, token_seq, query_start, context_lens, residual: bool, act: int = 0, in_bias=None,
+               bias1=None):
     """x [T, channels]; w1 / w2 [channels, taps] float32 (w2 may be None); history [slots, >= (taps - 1) channels] float32 is read
     and rewritten.  Returns (out1, out2 or None)."""
     from ._lib import TapFilterArgs
@@ -464,6 +465,7 @@ def tap_filter(x, w1, w2, history, state_slots, token_seq, query_start, context_
     a.history, a.history_stride = _p(history), 0 if history is None else history.stride(0)
     a.state_slots, a.token_seq, a.query_start, a.context_lens = _p(state_slots), _p(token_seq), _p(query_start), _p(context_lens)
     a.T, a.B, a.channels, a.taps, a.residual, a.act, a.dtype = T, context_lens.numel(), Cn, w1.shape[1], int(residual), act, _CODES[x.dtype]
+    a.in_bias, a.bias1 = _p(in_bias), _p(bias1)
     _lib.lib().atoma_tap_filter(C.byref(a), _s())
     _check()
     return out1, out2
@@ -509,7 +511,7 @@ def headnorm_gate(o, weight, gate, H, vdim, eps, dtype):
 
 
 def qkv_headnorm_rope_cache(proj, q_off, k_off, v_off, q_w, k_w, qk_freq, v_freq, interleaved, positions, slots, k_cache, v_cache, H, G,
-                            dim, vdim, eps):
+                            dim, vdim, eps, bias=None, q_head_scale=None, unit_norm=False):
     from ._lib import QkvRopeArgs
     T = proj.shape[0]
     q = torch.empty((T, H * dim), dtype=proj.dtype, device=proj.device)
@@ -519,6 +521,7 @@ def qkv_headnorm_rope_cache(proj, q_off, k_off, v_off, q_w, k_w, qk_freq, v_freq
     a.rot_pairs, a.v_pairs, a.interleaved = 0 if qk_freq is None else qk_freq.numel(), 0 if v_freq is None else v_freq.numel(), int(interleaved)
     a.positions, a.slot_mapping, a.q_out, a.k_cache, a.v_cache = _p(positions), _p(slots), _p(q), _p(k_cache), _p(v_cache)
     a.T, a.H, a.G, a.dim, a.vdim, a.eps, a.dtype = T, H, G, dim, vdim, eps, _CODES[proj.dtype]
+    a.bias, a.q_head_scale, a.unit_norm = _p(bias), _p(q_head_scale), int(unit_norm)
     _lib.lib().atoma_qkv_headnorm_rope_cache(C.byref(a), _s())
     _check()
     return q
@@ -531,28 +534,76 @@ def rotate_heads(x, positions, freq, H, n, interleaved, sign):
     return x
 
 
-def latent_norm_rope_cache(proj, q_weight, kv_weight, freq, interleaved, positions, slots, cache, q_rank, kv_rank, rot_dim, eps):
+def latent_norm_rope_cache(proj, q_weight, kv_weight, freq, interleaved, positions, slots, cache, q_rank, kv_rank, rot_dim, eps, freq_lo=None,
+                           amplitude=1.0):
     T = proj.shape[0]
     cq = torch.empty((T, q_rank), dtype=proj.dtype, device=proj.device)
-    _lib.lib().atoma_latent_norm_rope_cache(_p(proj), proj.stride(0), _p(q_weight), _p(kv_weight), _p(freq), 0 if freq is None else freq.numel(),
+    _lib.lib().atoma_latent_norm_rope_cache(_p(proj), proj.stride(0), _p(q_weight), _p(kv_weight), _p(freq), _p(freq_lo), amplitude,
+                                            0 if freq is None else freq.numel(),
                                             int(interleaved), _p(positions), _p(slots), _p(cq), _p(cache), T, q_rank, kv_rank, rot_dim, eps,
                                             _CODES[proj.dtype], _s())
     _check()
     return cq
 
 
-def latent_query_absorb_rope(q, w_uk, freq, interleaved, positions, H, dim, rot_dim, kv_rank):
+def latent_query_absorb_rope(q, w_uk, freq, interleaved, positions, H, dim, rot_dim, kv_rank, freq_lo=None, amplitude=1.0):
     T = q.shape[0]
     out = torch.empty((T, H, kv_rank + rot_dim), dtype=torch.float32, device=q.device)
-    _lib.lib().atoma_latent_query_absorb_rope(_p(q), _p(w_uk), _p(freq), 0 if freq is None else freq.numel(), int(interleaved), _p(positions),
+    _lib.lib().atoma_latent_query_absorb_rope(_p(q), _p(w_uk), _p(freq), _p(freq_lo), amplitude, 0 if freq is None else freq.numel(),
+                                              int(interleaved), _p(positions),
                                               _p(out), T, H, dim, rot_dim, kv_rank, _CODES[q.dtype], _s())
     _check()
     return out
 
 
-def latent_expand_values(o_lat, w_uv, H, vdim, kv_rank, dtype):
+def latent_expand_values(o_lat, w_uv, H, vdim, kv_rank, dtype, gate=None):
     T, row = o_lat.shape[0], o_lat.shape[-1]
     out = torch.empty((T, H * vdim), dtype=dtype, device=o_lat.device)
-    _lib.lib().atoma_latent_expand_values(_p(o_lat), _p(w_uv), _p(out), T, H, vdim, kv_rank, row, _CODES[dtype], _s())
+    _lib.lib().atoma_latent_expand_values(_p(o_lat), _p(w_uv), _p(gate), 0 if gate is None else gate.stride(0), _p(out), T, H, vdim, kv_rank, row, _CODES[dtype], _s())
+    _check()
+    return out
+
+
+def postnorm_residual(x, w_norm, alpha, eps, dtype, y=None, experts=None, depth=None, depth_w=None, depth_n=0, want_trace=False, offset=0.0):
+    """x [T, W] float32 is updated in place: x <- norm(alpha x + y + expert rows), row depth_n - 1 of depth [.., T, W] is written and x becomes
+    the weighted sum of its first depth_n rows.  experts: (expert_out address, pair_row address, top_expert, keep-alive).  Returns (h, trace)."""
+    from ._lib import PostnormArgs
+    T, W = x.shape
+    h = torch.empty((T, W), dtype=dtype, device=x.device)
+    trace = torch.empty_like(x) if want_trace else None
+    a = PostnormArgs()
+    a.y, a.x, a.w_norm, a.depth, a.depth_w, a.depth_n, a.h, a.trace = _p(y), _p(x), _p(w_norm), _p(depth), _p(depth_w), depth_n, _p(h), _p(trace)
+    if experts is not None:
+        a.expert_out, a.pair_row, a.top_expert, a.top = experts[0], experts[1], _p(experts[2]), experts[2].shape[1]
+    a.T, a.width, a.alpha, a.eps, a.weight_offset, a.dtype = T, W, alpha, eps, offset, _CODES[dtype]
+    _lib.lib().atoma_postnorm_residual(C.byref(a), _s())
+    _check()
+    return h, trace
+
+
+def lru_gates(u, w, bias_r, bias_i, rate, blocks):
+    """u [T, C]; w [blocks, 2 n, n] -> (decay, input) float32 [T, C]."""
+    from ._lib import LruGatesArgs
+    T, Cn = u.shape
+    decay, inp = (torch.empty((T, Cn), dtype=torch.float32, device=u.device) for _ in range(2))
+    a = LruGatesArgs()
+    a.u, a.ld_u, a.w, a.bias_r, a.bias_i, a.rate, a.decay, a.input = _p(u), u.stride(0), _p(w), _p(bias_r), _p(bias_i), _p(rate), _p(decay), _p(inp)
+    a.T, a.channels, a.blocks, a.dtype = T, Cn, blocks, _CODES[u.dtype]
+    _lib.lib().atoma_lru_gates(C.byref(a), _s())
+    _check()
+    return decay, inp
+
+
+def linear_scan(decay, inp, gate, gate_bias, state, state_slots, query_start, context_lens, max_query_len, act=2):
+    """S <- decay S + inp per channel and sequence; returns S * act(gate + gate_bias) [T, C] in the gate's format; state [slots, >= C]."""
+    from ._lib import LinearScanArgs
+    T, Cn = decay.shape
+    out = torch.empty((T, Cn), dtype=gate.dtype, device=gate.device)
+    a = LinearScanArgs()
+    a.decay, a.input, a.gate, a.ld_gate, a.gate_bias, a.state, a.state_stride = (_p(decay), _p(inp), _p(gate), gate.stride(0), _p(gate_bias), _p(state),
+                                                                               state.stride(0))
+    a.state_slots, a.query_start, a.context_lens, a.out = _p(state_slots), _p(query_start), _p(context_lens), _p(out)
+    a.T, a.B, a.channels, a.act, a.max_query_len, a.dtype = T, context_lens.numel(), Cn, act, max_query_len, _CODES[gate.dtype]
+    _lib.lib().atoma_linear_scan(C.byref(a), _s())
     _check()
     return out

@@ -39,6 +39,14 @@
  * head), each result RMS-normed over the model width before the two are averaged — and a span of layers that
  * runs several times with the embedding added again and a per-pass vector at the start of every pass.
  *
+ * The fifth design is Mobunex: POST-NORM blocks (x <- norm(alpha x + sublayer(x)), the sublayer reads the stream itself, a norm's
+ * weight is one number), a depth average after every layer (what goes on is a learned weighted sum of the embedding output and of
+ * every layer's result so far), grouped softmax attention under a sliding window with projection biases, unweighted per-head q/k
+ * norms and a factor per head on the score, a recurrent block with a real-gated linear recurrent unit (short causal filter,
+ * block-diagonal gates, a decay per channel and token), latent attention with a rotated key part (YaRN-scaled frequencies) under a
+ * sliding window with a sigmoid gate on the heads' outputs, and a mixture of experts whose groups are ranked by the sum of their two
+ * best choice scores.
+ *
  * Conventions: row-major; `dtype` is the number format of activations, large weights and the caches:
  * 1 = bfloat16, 2 = float32 (true 32-bit arithmetic: no reduced-precision matrix mode).  Whatever the
  * dtype, the residual stream, norm statistics, attention scores and weights, recurrent state and all
@@ -382,13 +390,13 @@ void atoma_softmax_attention_paged(const atoma_softmax_attn_args *args, atoma_st
 
 /* Router with a restricted choice, float32.  z = w_router h over `outputs` router rows (experts, then identity experts);
  * s = softmax(z) (score_fn 1) or sigmoid(z) (0); choice score c = s + correction (NULL: none).  The outputs form `groups`
- * equal groups of neighbours (groups <= 1: no restriction); a group's score is its largest c; only outputs of the `keep`
- * best groups can be chosen (ties: the lower group).  The `top` largest c among them (ties: the lower index) ->
+ * equal groups of neighbours (groups <= 1: no restriction); a group's score is the sum of its `group_top` largest c (1 or 2; a
+ * group of one output has only that one); only outputs of the `keep` best groups can be chosen (ties: the lower group).  The `top` largest c among them (ties: the lower index) ->
  * top_expert [T, top] (an index >= the caller's expert count is an identity expert; -1 where fewer than `top` could be
  * chosen) and top_weight = their s divided by (their sum + 1e-20) (renormalize 1) or as they are (0). */
 void atoma_moe_route_grouped(const void *h, const float *w_router, const float *correction, int32_t *top_expert, float *top_weight,
-                             int64_t T, int64_t width, int64_t outputs, int64_t top, int64_t groups, int64_t keep, int32_t score_fn,
-                             int32_t renormalize, uint32_t dtype, atoma_stream_t stream);
+                             int64_t T, int64_t width, int64_t outputs, int64_t top, int64_t groups, int64_t keep, int32_t group_top,
+                             int32_t score_fn, int32_t renormalize, uint32_t dtype, atoma_stream_t stream);
 
 /* act_out[T, ff] = clamped gated activation (atoma_glu_clamped_bias) of the projection x [T, K] w_gate_up [2 ff, K]^T (gate rows,
  * then up rows).  Decode-sized bfloat16 steps (T <= 128, K % 64 == 0) run ONE kernel, the activation in the tcgen05 product's
@@ -435,6 +443,8 @@ void atoma_parallel_residual_norm(const atoma_parallel_residual_args *args, atom
  * (w2 / out2 may be NULL: one filter).  For token t of sequence b at position p:
  *   f_k(t, c) = sum_{j < taps} w_k[c, j] * in(position p - (taps - 1) + j, c)       zero before the sequence's start
  *   out_k[t, c] = act(residual ? in[t, c] + f_k : f_k)        act: 0 = none, 1 = silu        (`dtype`, row stride ld_out)
+ * in_bias [channels] (NULL: none) is part of the input: in(.) above is the stored value plus in_bias for every token of the
+ * sequence (zero before its start, without the bias), and the history keeps the sum.  bias1 [channels] (NULL: none) is added to f_1.
  * history [slots, history_stride] float32 holds, at the slot of the sequence, its last taps - 1 inputs as
  * [taps - 1, channels]; it is read for positions before the portion (never when they lie before the sequence's start)
  * and rewritten with the portion's last inputs.  taps <= 16.
@@ -454,6 +464,7 @@ typedef struct atoma_tap_filter_args {
     int64_t T, B, channels, taps;
     int32_t residual, act;
     uint32_t dtype;
+    const float *in_bias, *bias1; /* [channels] or NULL */
 } atoma_tap_filter_args;
 void atoma_tap_filter(const atoma_tap_filter_args *args, atoma_stream_t stream);
 
@@ -495,6 +506,8 @@ void atoma_headnorm_gate(const float *o, const float *weight, const void *gate, 
  * at v_off (G of vdim).  Per head: RMS norm over dim with q_weight / k_weight ([dim], NULL: none), then the first
  * 2 rot_pairs entries are turned by position * qk_freq[i] (float32 angle) in pairs (2i, 2i + 1) (interleaved = 1) or
  * (i, i + rot_pairs) (0); the values' first 2 v_pairs entries likewise by v_freq (v_freq NULL: stored as projected).
+ * bias (float32, indexed by the columns of proj; NULL: none) is added to the projections first; unit_norm 1 divides every query
+ * and key head by its root mean square also without a weight; q_head_scale [H] (NULL: none) multiplies a normed query head.
  * q -> q_out [T, H dim]; k, v -> cache rows slot_mapping[t] (slot < 0 is skipped).
  */
 typedef struct atoma_qkv_rope_args {
@@ -509,6 +522,8 @@ typedef struct atoma_qkv_rope_args {
     int64_t T, H, G, dim, vdim;
     float eps;
     uint32_t dtype;
+    const float *bias, *q_head_scale;
+    int32_t unit_norm;
 } atoma_qkv_rope_args;
 void atoma_qkv_headnorm_rope_cache(const atoma_qkv_rope_args *args, atoma_stream_t stream);
 
@@ -519,30 +534,107 @@ void atoma_rotate_heads(void *x, const int64_t *positions, const float *freq, in
 /*
  * Latent attention with a rotated key part.  proj[t, :] (row stride ld) = [c_q (q_rank) | c (kv_rank) | k_rot (rot_dim)]:
  *   cq_out[t, :] = rms(c_q) * q_weight;   cache[slot_mapping[t], :] = [rms(c) * kv_weight | rotate(k_rot, position)]
- * rotation in pairs (i, i + pairs) (interleaved 0) or (2i, 2i + 1); cache rows of kv_rank + rot_dim in `dtype`.
+ * rotation in pairs (i, i + pairs) (interleaved 0) or (2i, 2i + 1) by position * (freq[i] + freq_lo[i]) (freq_lo: what float32 drops
+ * of the frequency, NULL: none; the product is formed to twice float32's precision), cos and sin times `amplitude`; cache rows of
+ * kv_rank + rot_dim in `dtype`.
  */
 void atoma_latent_norm_rope_cache(const void *proj, int64_t ld, const float *q_weight, const float *kv_weight, const float *freq,
-                                  int64_t pairs, int32_t interleaved, const int64_t *positions, const int64_t *slot_mapping,
+                                  const float *freq_lo, float amplitude, int64_t pairs, int32_t interleaved, const int64_t *positions, const int64_t *slot_mapping,
                                   void *cq_out, void *cache, int64_t T, int64_t q_rank, int64_t kv_rank, int64_t rot_dim, float eps,
                                   uint32_t dtype, atoma_stream_t stream);
 
 /* Queries q [T, H, dim + rot_dim] (`dtype`) into the space of the cached rows, q_lat float32 [T, H, kv_rank + rot_dim]:
  *   q_lat[t, h, :kv_rank] = w_uk_h^T q[t, h, :dim]  (w_uk [H dim, kv_rank]);   q_lat[t, h, kv_rank:] = rotate(q[t, h, dim:], position) */
-void atoma_latent_query_absorb_rope(const void *q, const void *w_uk, const float *freq, int64_t pairs, int32_t interleaved,
-                                    const int64_t *positions, float *q_lat, int64_t T, int64_t H, int64_t dim, int64_t rot_dim,
+void atoma_latent_query_absorb_rope(const void *q, const void *w_uk, const float *freq, const float *freq_lo, float amplitude, int64_t pairs,
+                                    int32_t interleaved, const int64_t *positions, float *q_lat, int64_t T, int64_t H, int64_t dim, int64_t rot_dim,
                                     int64_t kv_rank, uint32_t dtype, atoma_stream_t stream);
 
 /* Values of every head from its weighted sum of cached rows: out[t, h vdim + j] = sum_{r < kv_rank} o_lat[t, h, r] w_uv[h vdim + j, r];
- * o_lat float32 [T, H, row] with row >= kv_rank (what lies behind kv_rank is not read). */
-void atoma_latent_expand_values(const float *o_lat, const void *w_uv, void *out, int64_t T, int64_t H, int64_t vdim, int64_t kv_rank,
-                                int64_t row, uint32_t dtype, atoma_stream_t stream);
+ * o_lat float32 [T, H, row] with row >= kv_rank (what lies behind kv_rank is not read).  gate (row stride ld_gate, `dtype`, NULL:
+ * none): the result times sigmoid(gate[t, h vdim + j]). */
+void atoma_latent_expand_values(const float *o_lat, const void *w_uv, const void *gate, int64_t ld_gate, void *out, int64_t T, int64_t H,
+                                int64_t vdim, int64_t kv_rank, int64_t row, uint32_t dtype, atoma_stream_t stream);
+
+/* ------------------------------------------------------------------------------------------ */
+/* Post-norm blocks with a depth average; real-gated linear recurrent unit                      */
+/* ------------------------------------------------------------------------------------------ */
+
+/*
+ * Residual update of a post-norm block, fused with the sum of the token's expert rows and the average over depth.  Per token t:
+ *   v = alpha * x[t, :] + (y ? y[t, :] : 0) + sum_{k < top} (top_expert[t, k] >= 0: expert_out[pair_row[t top + k], :])
+ *   n = v / sqrt(mean(v^2) + eps) * (weight_offset + w_norm)
+ *   x[t, :] = n                                                              (depth_n = 0)
+ *   depth[depth_n - 1][t, :] = n;  x[t, :] = sum_{j < depth_n} depth_w[j] depth[j][t, :]   (depth_n > 0; depth_w NULL: x = n)
+ *   h[t, :] = x[t, :] in `dtype` (NULL: not written);   trace[t, :] = x[t, :] (NULL: not written)
+ * x float32 [T, width] in place; depth float32 [.., T, width] (row j of the average at j T width), rows 0 .. depth_n - 2 written by
+ * earlier calls.  y, expert_out, h in `dtype`.  Experts' rows are added in the order of k, depth rows in the order of j.
+ */
+typedef struct atoma_postnorm_args {
+    const void *y;
+    const void *expert_out;
+    const int32_t *pair_row;      /* [T top] */
+    const int32_t *top_expert;    /* [T top] (NULL with expert_out: every pair has a row) */
+    int64_t top;
+    float *x;
+    const float *w_norm;          /* [width] */
+    float *depth;
+    const float *depth_w;         /* [depth_n] or NULL */
+    int64_t depth_n;
+    void *h;
+    float *trace;
+    int64_t T, width;
+    float alpha, eps, weight_offset;
+    uint32_t dtype;
+} atoma_postnorm_args;
+void atoma_postnorm_residual(const atoma_postnorm_args *args, atoma_stream_t stream);
+
+/*
+ * Gates of a real-gated linear recurrent unit with block-diagonal gate matrices.  u [T, channels] (`dtype`, row stride ld_u) in
+ * `blocks` equal parts of n = channels / blocks; w [blocks, 2 n, n] `dtype` (a part's first n rows make the recurrence gate r, the next
+ * n the input gate i, stored [out, in]); bias_r, bias_i, rate [channels] float32.  Everything behind the products is float32:
+ *   r = sigmoid(w_r u + bias_r);  i = sigmoid(w_i u + bias_i);  log a = rate * r  (rate <= 0)
+ *   decay[t, c] = exp(log a);     input[t, c] = sqrt(1 - a^2) * i * u[t, c]        (1 - a^2 without cancellation)
+ * decay and input float32 [T, channels].
+ */
+typedef struct atoma_lru_gates_args {
+    const void *u;
+    int64_t ld_u;
+    const void *w;
+    const float *bias_r, *bias_i, *rate;
+    float *decay, *input;
+    int64_t T, channels, blocks;
+    uint32_t dtype;
+} atoma_lru_gates_args;
+void atoma_lru_gates(const atoma_lru_gates_args *args, atoma_stream_t stream);
+
+/*
+ * Linear recurrence with one float32 state per channel on a mixed batch: per sequence, in token order,
+ *   S <- decay[t, c] S + input[t, c];   out[t, c] = S * act(gate[t, c] + gate_bias[c])        act: 0 silu, 1 relu, 2 gelu (tanh form)
+ * S starts from state[state_slots[b], c] — from zero when context_lens[b] == 0 — and is stored back.  decay, input float32
+ * [T, channels]; gate (row stride ld_gate) and out [T, channels] in `dtype`; state rows state_stride floats apart.
+ */
+typedef struct atoma_linear_scan_args {
+    const float *decay, *input;
+    const void *gate;
+    int64_t ld_gate;
+    const float *gate_bias;       /* [channels] or NULL */
+    float *state;
+    int64_t state_stride;
+    const int32_t *state_slots, *query_start, *context_lens;
+    void *out;
+    int64_t T, B, channels;
+    int32_t act, max_query_len;
+    uint32_t dtype;
+} atoma_linear_scan_args;
+void atoma_linear_scan(const atoma_linear_scan_args *args, atoma_stream_t stream);
 
 /* ------------------------------------------------------------------------------------------ */
 /* Step executor                                                                                */
 /* ------------------------------------------------------------------------------------------ */
 enum { ATOMA_MIXER_SIGMOID_ATTENTION = 0, ATOMA_MIXER_MINGRU = 1, ATOMA_MIXER_LATENT_ATTENTION = 2, ATOMA_MIXER_SOFTMAX_ATTENTION = 3,
-       ATOMA_MIXER_GLA = 4, ATOMA_MIXER_PAIR = 5 };
-enum { ATOMA_BLOCK_SANDWICH = 0, ATOMA_BLOCK_PRENORM = 1, ATOMA_BLOCK_LANES = 2, ATOMA_BLOCK_PARALLEL = 3 };
+       ATOMA_MIXER_GLA = 4, ATOMA_MIXER_PAIR = 5, ATOMA_MIXER_LRU = 6 };
+enum { ATOMA_BLOCK_SANDWICH = 0, ATOMA_BLOCK_PRENORM = 1, ATOMA_BLOCK_LANES = 2, ATOMA_BLOCK_PARALLEL = 3,
+       ATOMA_BLOCK_POSTNORM = 4 };
 enum { ATOMA_SCORE_SIGMOID = 0, ATOMA_SCORE_SOFTMAX = 1 };
 enum { ATOMA_FF_DENSE = 0, ATOMA_FF_MOE = 1 };
 enum { ATOMA_ACT_SILU = 0, ATOMA_ACT_RELU = 1, ATOMA_ACT_GELU_TANH = 2 };
@@ -634,6 +726,21 @@ typedef struct atoma_hybrid_layer {
     /* latent attention with a rotated key part (q_rank, kv_rank, dq_norm, dkv_norm, w_uq [heads (dim + rot_dim), q_rank], w_uk, w_uv,
      * latent_cache rows of kv_rank + rot_dim; qk_freq / rot_pairs / rot_interleaved above) */
     int64_t rot_dim;
+    /* ---- post-norm blocks (model.block_style = ATOMA_BLOCK_POSTNORM): x <- norm(alpha x + sublayer(x)) ---- */
+    /* norm1 / norm2 above follow the sums; b_qkv [proj_cols] = biases of the stacked projection; softmax attention: columns q_off, k_off,
+     * v_off; latent attention: [c_q | c | k_rot] at column 0, the output gate's pre-activation at g_off (out_gate); mixture of experts:
+     * w_ff_in = the shared expert's gate and up rows */
+    const float *depth_w;            /* weights of the embedding output and of every layer's result up to this one, or NULL */
+    const float *q_head_scale;       /* [heads] or NULL */
+    const float *qk_freq_lo;         /* [rot_pairs] or NULL */
+    float rot_amplitude;
+    int32_t route_group_top;         /* choice scores of a group that make its score (1 or 2; 0 = 1) */
+    /* real-gated linear recurrent unit: width lru_width, gate branch at column q_off, recurrent branch at k_off, filter r_tap_w
+     * [lru_width, r_taps] with bias; the layer's state row = [filter history (r_taps - 1) lru_width | state lru_width] */
+    int64_t lru_width, lru_blocks;
+    const void *lru_w;               /* [lru_blocks, 2 n, n] */
+    const float *lru_bias_r, *lru_bias_i, *lru_rate, *r_tap_bias; /* [lru_width] */
+    const void *w_uk_rot;            /* [heads (dim + rot_dim), kv_rank + rot_dim]: a cached row -> the heads' whole keys, or NULL */
 } atoma_hybrid_layer;
 
 typedef struct atoma_hybrid_model {
@@ -656,6 +763,9 @@ typedef struct atoma_hybrid_model {
     /* ---- designs on residual lanes ---- */
     int32_t lanes;          /* copies of the residual stream (ATOMA_BLOCK_LANES: >= 1) */
     float embed_scale;      /* the embedding row times this; no position signal is added */
+    /* ---- post-norm designs ---- */
+    const float *embed_norm; /* [width]: norm of the embedding rows */
+    float residual_alpha;   /* the stream's factor in every sum */
 } atoma_hybrid_model;
 
 typedef struct atoma_hybrid_batch {
@@ -681,7 +791,7 @@ typedef struct atoma_hybrid_batch {
     int64_t long_tokens, long_ctx_sum;
 } atoma_hybrid_batch;
 
-int64_t atoma_hybrid_abi_sizeof(int which); /* 0 layer, 1 model, 2 batch, 3 attention args, 4 gated residual args, 5 latent attention args, 6 expert args, 7 expanded attention args, 8 lanes update args, 9 softmax attention args, 10 parallel residual args, 11 tap filter args, 12 state scan args, 13 rotary cache args */
+int64_t atoma_hybrid_abi_sizeof(int which); /* 0 layer, 1 model, 2 batch, 3 attention args, 4 gated residual args, 5 latent attention args, 6 expert args, 7 expanded attention args, 8 lanes update args, 9 softmax attention args, 10 parallel residual args, 11 tap filter args, 12 state scan args, 13 rotary cache args, 14 post-norm args, 15 gate args, 16 linear scan args */
 int64_t atoma_hybrid_scratch_bytes(const atoma_hybrid_model *model, int64_t num_tokens, int64_t num_selected);
 void atoma_hybrid_step(const atoma_hybrid_model *model, const atoma_hybrid_batch *batch, atoma_stream_t stream);
 
