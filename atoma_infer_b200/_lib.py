@@ -326,7 +326,8 @@ class LatentExpandedArgs(C.Structure):
 
     _fields_ = ([(n, C.c_void_p) for n in ("q", "latent_cache", "w_uk", "w_uv", "out", "query_start", "context_lens", "block_tables", "sink")] +
                 [(n, C.c_int64) for n in ("T", "B", "max_blocks", "H", "dim", "R", "block_size", "window", "max_keys")] +
-                [("scale", C.c_float), ("min_q", C.c_int32), ("max_query_len", C.c_int32), ("max_seq_len", C.c_int32)])
+                [("scale", C.c_float), ("min_q", C.c_int32), ("max_query_len", C.c_int32), ("max_seq_len", C.c_int32), ("rot_dim", C.c_int64),
+                 ("vdim", C.c_int64), ("gate", C.c_void_p), ("ld_gate", C.c_int64)])
 
 
 class MoeArgs(C.Structure):
@@ -483,7 +484,7 @@ SIGNATURES = {
     "atoma_state_scan": (None, [C.POINTER(StateScanArgs), C.c_void_p]),
     "atoma_headnorm_gate": (None, [C.c_void_p] * 3 + [C.c_int64, C.c_void_p] + [C.c_int64] * 3 + [C.c_float, C.c_uint32, C.c_void_p]),
     "atoma_qkv_headnorm_rope_cache": (None, [C.POINTER(QkvRopeArgs), C.c_void_p]),
-    "atoma_rotate_heads": (None, [C.c_void_p] * 3 + [C.c_int64] * 4 + [C.c_int32, C.c_float, C.c_uint32, C.c_void_p]),
+    "atoma_rotate_heads": (None, [C.c_void_p] * 4 + [C.c_float] + [C.c_int64] * 4 + [C.c_int32, C.c_float, C.c_uint32, C.c_void_p]),
     "atoma_latent_norm_rope_cache": (None, [C.c_void_p, C.c_int64] + [C.c_void_p] * 4 + [C.c_float, C.c_int64, C.c_int32] + [C.c_void_p] * 4 +
                                      [C.c_int64] * 4 + [C.c_float, C.c_uint32, C.c_void_p]),
     "atoma_latent_query_absorb_rope": (None, [C.c_void_p] * 4 + [C.c_float, C.c_int64, C.c_int32, C.c_void_p, C.c_void_p] + [C.c_int64] * 5 +
@@ -496,6 +497,7 @@ SIGNATURES = {
     "atoma_hybrid_scratch_bytes": (C.c_int64, [C.POINTER(HybridModel), C.c_int64, C.c_int64]),
     "atoma_hybrid_step": (None, [C.POINTER(HybridModel), C.POINTER(HybridBatch), C.c_void_p]),
     "atoma_debug_hybrid": (None, [C.c_int]),
+    "atoma_prefill_timeouts": (C.c_int, []),
     # atoma_ops.h
     "atoma_flash_attn_plan": (C.c_char_p, [C.POINTER(Tensor)] * 4 + [C.c_float, C.c_int64, C.c_int64, C.c_float,
                                                                     C.c_int, C.POINTER(MhaPlan)]),

@@ -45,7 +45,7 @@ bool hyb_latent_norm_cache(const void *, int64_t, const float *, const float *, 
                            float, uint32_t, cudaStream_t);
 bool hyb_head_project(const void *, const void *, void *, int64_t, int64_t, int64_t, int64_t, int32_t, uint32_t, cudaStream_t);
 bool hyb_latent_attention(const atoma_latent_attn_args &, cudaStream_t);
-bool hyb_latent_expanded_ok(int64_t, int64_t, int64_t, uint32_t);
+bool hyb_latent_expanded_ok(int64_t, int64_t, int64_t, int64_t, uint32_t);
 bool hyb_latent_attention_expanded(const atoma_latent_expanded_args &, cudaStream_t);
 bool hyb_moe_route(const void *, const float *, const float *, int32_t *, float *, float *, int64_t, int64_t, int64_t, int64_t, int32_t,
                    uint32_t, cudaStream_t);
@@ -66,7 +66,7 @@ bool hyb_tap_filter(const atoma_tap_filter_args &, cudaStream_t);
 bool hyb_state_scan(const atoma_state_scan_args &, cudaStream_t);
 bool hyb_headnorm_gate(const float *, const float *, const void *, int64_t, void *, int64_t, int64_t, int64_t, float, uint32_t, cudaStream_t);
 bool hyb_qkv_headnorm_rope_cache(const atoma_qkv_rope_args &, cudaStream_t);
-bool hyb_rotate_heads(void *, const int64_t *, const float *, int64_t, int64_t, int64_t, int64_t, int32_t, float, uint32_t, cudaStream_t);
+bool hyb_rotate_heads(void *, const int64_t *, const float *, const float *, float, int64_t, int64_t, int64_t, int64_t, int32_t, float, uint32_t, cudaStream_t);
 bool hyb_latent_norm_rope_cache(const void *, int64_t, const float *, const float *, const float *, const float *, float, int64_t, int32_t,
                                 const int64_t *, const int64_t *, void *, void *, int64_t, int64_t, int64_t, int64_t, float, uint32_t, cudaStream_t);
 bool hyb_latent_query_absorb_rope(const void *, const void *, const float *, const float *, float, int64_t, int32_t, const int64_t *, float *, int64_t,
@@ -284,7 +284,7 @@ bool prenorm_layer(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, con
     if (!hyb_linear(s.cq, l.w_uq, s.q, T, l.heads * l.dim, l.q_rank, dt, stream)) return false;
     // long prompt portions run on expanded keys and values (4x fewer multiply-adds per pair at usual sizes); decoded tokens and
     // short portions run in the latent space (the cache is read once for all heads)
-    const bool expanded = b.long_seqs > 0 && b.long_min_q >= 32 && hyb_latent_expanded_ok(l.dim, l.vdim, l.kv_rank, dt);
+    const bool expanded = b.long_seqs > 0 && b.long_min_q >= 32 && l.dim == l.vdim && hyb_latent_expanded_ok(l.dim, 0, l.vdim, l.kv_rank, dt);
     const bool latent_too = !expanded || b.long_seqs < b.num_seqs;
     if (latent_too && !hyb_head_project(s.q, l.w_uk, s.qlat, T, l.heads, l.dim, l.kv_rank, 1, dt, stream)) return false;
     atoma_latent_attn_args a{};
@@ -736,7 +736,7 @@ bool parallel_layer(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, co
         a.dtype = dt;
         a.max_query_len = b.max_query_len;
         if (!hyb_attention(a, stream)) return false;
-        if (l.v_freq && !hyb_rotate_heads(s.act, b.positions, l.v_freq, T, l.heads, l.vdim, l.v_pairs, l.rot_interleaved, -1.f, dt, stream))
+        if (l.v_freq && !hyb_rotate_heads(s.act, b.positions, l.v_freq, nullptr, 1.f, T, l.heads, l.vdim, l.v_pairs, l.rot_interleaved, -1.f, dt, stream))
             return false;
         if (!hyb_linear(s.act, l.w_o, s.y, T, W, l.heads * l.vdim, dt, stream)) return false;
         // right: gated delta rule behind short filters
@@ -882,32 +882,70 @@ bool postnorm_latent(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, c
                                     b.positions, b.slot_mapping, s.cq, l.latent_cache, T, l.q_rank, l.kv_rank, l.rot_dim, m.eps, dt, stream))
         return false;
     if (!hyb_linear(s.cq, l.w_uq, s.q, T, H * (l.dim + l.rot_dim), l.q_rank, dt, stream)) return false;
-    if (!hyb_latent_query_absorb_rope(s.q, l.w_uk, l.qk_freq, l.qk_freq_lo, l.rot_amplitude, l.rot_pairs, l.rot_interleaved, b.positions, s.qlat,
-                                      T, H, l.dim, l.rot_dim, l.kv_rank, dt, stream))
+    // long prompt portions run on expanded keys and values, decoded tokens and short portions in the space of the cached rows
+    const bool expanded = b.long_seqs > 0 && b.long_min_q >= 32 && l.w_uk_rot && hyb_latent_expanded_ok(l.dim, l.rot_dim, l.vdim, l.kv_rank, dt);
+    if (!expanded || b.long_seqs < b.num_seqs) {
+        if (!hyb_latent_query_absorb_rope(s.q, l.w_uk, l.qk_freq, l.qk_freq_lo, l.rot_amplitude, l.rot_pairs, l.rot_interleaved, b.positions, s.qlat,
+                                          T, H, l.dim, l.rot_dim, l.kv_rank, dt, stream))
+            return false;
+        atoma_latent_attn_args a{};
+        a.q_lat = s.qlat;
+        a.latent_cache = l.latent_cache;
+        a.out = s.olat;
+        a.positions = b.positions;
+        a.token_seq = b.token_seq;
+        a.query_start = b.query_start;
+        a.block_tables = b.block_tables;
+        a.sink = l.sink;
+        a.T = T;
+        a.B = b.num_seqs;
+        a.max_blocks = b.max_blocks;
+        a.H = H;
+        a.R = row;
+        a.block_size = m.block_size;
+        a.window = l.window;
+        a.scale = l.scale;
+        a.dtype = dt;
+        a.max_query_len = b.max_query_len;
+        a.max_seq_len = b.max_seq_len;
+        a.skip_min_q = expanded ? b.long_min_q : 0;
+        a.out_cols = l.kv_rank;            // the rotated tail of a cached row takes part in the scores only
+        if (!hyb_latent_attention(a, stream)) return false;
+        if (!hyb_latent_expand_values(s.olat, l.w_uv, gate, P, s.act, T, H, l.vdim, l.kv_rank, row, dt, stream)) return false;
+    }
+    if (!expanded) return true;
+    // after the path above: it rewrites the long sequences' rows of s.act, and the queries are turned in place
+    if (l.rot_pairs > 0 && !hyb_rotate_heads(s.q + l.dim * es, b.positions, l.qk_freq, l.qk_freq_lo, l.rot_amplitude, T, H, l.dim + l.rot_dim, l.rot_pairs,
+                                             l.rot_interleaved, 1.f, dt, stream))
         return false;
-    atoma_latent_attn_args a{};
-    a.q_lat = s.qlat;
-    a.latent_cache = l.latent_cache;
-    a.out = s.olat;
-    a.positions = b.positions;
-    a.token_seq = b.token_seq;
-    a.query_start = b.query_start;
-    a.block_tables = b.block_tables;
-    a.sink = l.sink;
-    a.T = T;
-    a.B = b.num_seqs;
-    a.max_blocks = b.max_blocks;
-    a.H = H;
-    a.R = row;
-    a.block_size = m.block_size;
-    a.window = l.window;
-    a.scale = l.scale;
-    a.dtype = dt;
-    a.max_query_len = b.max_query_len;
-    a.max_seq_len = b.max_seq_len;
-    a.out_cols = l.kv_rank;            // the rotated tail of a cached row takes part in the scores only
-    if (!hyb_latent_attention(a, stream)) return false;
-    return hyb_latent_expand_values(s.olat, l.w_uv, gate, P, s.act, T, H, l.vdim, l.kv_rank, row, dt, stream);
+    atoma_latent_expanded_args e{};
+    e.q = s.q;
+    e.latent_cache = l.latent_cache;
+    e.w_uk = l.w_uk_rot;
+    e.w_uv = l.w_uv;
+    e.out = s.act;
+    e.query_start = b.query_start;
+    e.context_lens = b.context_lens;
+    e.block_tables = b.block_tables;
+    e.sink = l.sink;
+    e.T = T;
+    e.B = b.num_seqs;
+    e.max_blocks = b.max_blocks;
+    e.H = H;
+    e.dim = l.dim;
+    e.R = l.kv_rank;
+    e.block_size = m.block_size;
+    e.window = l.window;
+    e.max_keys = b.long_tokens + (l.window > 0 ? std::min<int64_t>(b.long_ctx_sum, static_cast<int64_t>(b.long_seqs) * (l.window - 1)) : b.long_ctx_sum);
+    e.scale = l.scale;
+    e.min_q = b.long_min_q;
+    e.max_query_len = b.max_query_len;
+    e.max_seq_len = b.max_seq_len;
+    e.rot_dim = l.rot_dim;
+    e.vdim = l.vdim;
+    e.gate = gate;
+    e.ld_gate = P;
+    return hyb_latent_attention_expanded(e, stream);
 }
 
 // Recurrent block of a post-norm layer: short filter -> gates -> scan, times the activated gate branch -> s.act.

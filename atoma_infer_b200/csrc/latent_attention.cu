@@ -15,6 +15,7 @@
 #include "tc_products.cuh"
 
 #include "atoma_hybrid.h"
+#include "atoma_llama.h"
 
 #include <algorithm>
 #include <cstring>
@@ -758,28 +759,33 @@ bool hyb_latent_attention(const atoma_latent_attn_args &a, cudaStream_t stream) 
 }
 
 
-// Shapes the expanded path takes: bfloat16, equal key and value head sizes of 64 or 128, 16-byte latent rows, sm_100.
-bool hyb_latent_expanded_ok(int64_t dim, int64_t vdim, int64_t R, uint32_t dtype) {
-    return dtype == ATOMA_DTYPE_BF16 && dim == vdim && (dim == 64 || dim == 128) && R % 8 == 0 && current_device_info().cc_major == 10 &&
-           !(g_hybrid_debug & 2);
+// Shapes the expanded path takes: bfloat16, values of 64 or 128, keys (with their rotated part) of up to 64 more entries, 16-byte
+// rows, sm_100.
+bool hyb_latent_expanded_ok(int64_t dim, int64_t rot_dim, int64_t vdim, int64_t R, uint32_t dtype) {
+    const int64_t dk = dim + rot_dim;
+    return dtype == ATOMA_DTYPE_BF16 && (vdim == 64 || vdim == 128) && dk > 0 && dk % 8 == 0 && dk <= vdim + 64 && (R + rot_dim) % 8 == 0 && R % 8 == 0 &&
+           current_device_info().cc_major == 10 && !(g_hybrid_debug & 2);
 }
 
 bool hyb_latent_attention_expanded(const atoma_latent_expanded_args &a, cudaStream_t stream) {
     if (a.T <= 0 || a.B <= 0 || a.max_keys <= 0) return true;
+    const int64_t vdim = a.vdim > 0 ? a.vdim : a.dim, dk = a.dim + a.rot_dim, row = a.R + a.rot_dim;
+    auto al = [](const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
     if (!a.q || !a.latent_cache || !a.w_uk || !a.w_uv || !a.out || !a.query_start || !a.context_lens || !a.block_tables || a.H <= 0 ||
-        a.min_q < 32 || !hyb_latent_expanded_ok(a.dim, a.dim, a.R, ATOMA_DTYPE_BF16)) {
-        set_status(kErrInvalidArg, "atoma_latent_attention_expanded: null argument, or a shape outside bfloat16 heads of 64 / 128 with min_q >= 32");
+        a.min_q < 32 || a.rot_dim < 0 || !hyb_latent_expanded_ok(a.dim, a.rot_dim, vdim, a.R, ATOMA_DTYPE_BF16) || (a.gate && a.ld_gate < a.H * vdim) ||
+        !al(a.q) || !al(a.out) || !al(a.latent_cache) || !al(a.w_uk) || !al(a.w_uv)) {
+        set_status(kErrInvalidArg, "atoma_latent_attention_expanded: null or unaligned argument, or a shape outside bfloat16 values of 64 / 128 with min_q >= 32");
         return false;
     }
-    const int64_t HD = a.H * a.dim;
+    const int64_t HK = a.H * dk, HV = a.H * vdim;
     auto up = [](int64_t x) { return (x + 255) / 256 * 256; };
     const int64_t rows = a.max_keys + 128;   // the attention kernel's TMA boxes may start up to a tile before the end
-    const int64_t b_int = up((2 * a.B + 2) * 4), b_c = up(rows * a.R * 2), b_kv = up(rows * HD * 2);
-    char *ws = static_cast<char *>(get_workspace(stream, static_cast<size_t>(b_int + b_c + 2 * b_kv), kWorkspaceLatentExpand));
+    const int64_t b_int = up((2 * a.B + 2) * 4), b_c = up(rows * row * 2), b_k = up(rows * HK * 2), b_v = up(rows * HV * 2);
+    char *ws = static_cast<char *>(get_workspace(stream, static_cast<size_t>(b_int + b_c + b_k + b_v), kWorkspaceLatentExpand));
     if (!ws) return false;
     int32_t *cu_k = reinterpret_cast<int32_t *>(ws), *key_lo = cu_k + a.B + 1;
     __nv_bfloat16 *C = reinterpret_cast<__nv_bfloat16 *>(ws + b_int);
-    __nv_bfloat16 *K = reinterpret_cast<__nv_bfloat16 *>(ws + b_int + b_c), *V = reinterpret_cast<__nv_bfloat16 *>(ws + b_int + b_c + b_kv);
+    __nv_bfloat16 *K = reinterpret_cast<__nv_bfloat16 *>(ws + b_int + b_c), *V = reinterpret_cast<__nv_bfloat16 *>(ws + b_int + b_c + b_k);
     if (!hybrid::launched(launch_ex(latent_expand_plan_kernel, dim3(1), dim3(32), 0, stream, a.query_start, a.context_lens,
                                     static_cast<int>(a.B), static_cast<int>(a.window), static_cast<int>(a.min_q), cu_k, key_lo),
                           "latent_expand_plan_kernel"))
@@ -788,23 +794,25 @@ bool hyb_latent_attention_expanded(const atoma_latent_expanded_args &a, cudaStre
     const dim3 gg(static_cast<unsigned>((span + 7) / 8), static_cast<unsigned>(a.B));
     if (!hybrid::launched(launch_ex(latent_gather_kernel, gg, dim3(256), 0, stream, static_cast<const __nv_bfloat16 *>(a.latent_cache),
                                     a.block_tables, a.max_blocks, static_cast<const int32_t *>(cu_k), static_cast<const int32_t *>(key_lo), C,
-                                    static_cast<int>(a.R), static_cast<int>(a.block_size)),
+                                    static_cast<int>(row), static_cast<int>(a.block_size)),
                           "latent_gather_kernel"))
         return false;
-    if (!hyb_linear(C, a.w_uk, K, a.max_keys, HD, a.R, ATOMA_DTYPE_BF16, stream)) return false;
-    if (!hyb_linear(C, a.w_uv, V, a.max_keys, HD, a.R, ATOMA_DTYPE_BF16, stream)) return false;
+    if (!hyb_linear(C, a.w_uk, K, a.max_keys, HK, row, ATOMA_DTYPE_BF16, stream)) return false;
+    atoma_gemm_tn(C, a.w_uv, V, a.max_keys, HV, a.R, row, a.R, HV, 1, stream);   // the values ignore the rows' tail
+    if (atoma_last_status() != 0) return false;
     MhaParams p;
     std::memset(&p, 0, sizeof(p));
     p.q = a.q, p.k = K, p.v = V, p.o = a.out;
     p.cu_q = a.query_start, p.cu_k = cu_k;
-    p.q_rs = p.k_rs = p.v_rs = p.o_rs = HD;
-    p.q_hs = p.k_hs = p.v_hs = p.o_hs = a.dim;
-    p.b = static_cast<int>(a.B), p.h = p.h_k = static_cast<int>(a.H), p.d = static_cast<int>(a.dim);
+    p.q_rs = p.k_rs = HK, p.v_rs = p.o_rs = HV;
+    p.q_hs = p.k_hs = dk, p.v_hs = p.o_hs = vdim;
+    p.b = static_cast<int>(a.B), p.h = p.h_k = static_cast<int>(a.H), p.d = static_cast<int>(vdim), p.d_k = static_cast<int>(dk);
     p.seqlen_q = a.max_query_len, p.seqlen_k = static_cast<int>(span);
     p.page = 1;
     p.scale = a.scale, p.scale_log2 = a.scale * 1.4426950408889634f;
     p.is_causal = 1, p.k_cumulative = 1;
     p.window_left = static_cast<int>(a.window), p.min_len_q = a.min_q, p.sink = a.sink;
+    p.gate = a.gate, p.gate_rs = a.ld_gate;
     const int r = try_launch_prefill_tc(p, true, stream);
     if (r == 1) return true;
     if (r == 0) set_status(kErrUnsupported, "atoma_latent_attention_expanded: the step is outside the tensor-memory attention kernel's envelope");

@@ -42,6 +42,11 @@ struct MhaParams {
     // added to the scaled score
     const float *dist_bias;
     int dist_rows, dist_heads;
+    // tcgen05 prefill kernel only: entries of a query / key head when they differ from the value head's d (0: the same), and a gate on the
+    // outputs (null = none): out times sigmoid(gate[(first row of the sequence + i) * gate_rs + head * d + c]), rows as cu_q counts them
+    int d_k;
+    const void *gate;
+    int64_t gate_rs;
 };
 
 }  // namespace atoma

@@ -548,8 +548,9 @@ __device__ __forceinline__ void turn(float pos, float freq, float freq_lo, float
     const float rest = fmaf(pos, freq, -ang) + pos * freq_lo;
     float s, c;
     sincosf(ang, &s, &c);
-    sn = amplitude * fmaf(rest, c, s);
-    cs = amplitude * fmaf(-rest, s, c);
+    const float near_one = fmaf(-0.5f * rest, rest, 1.f);     // cos of the correction; its sine is the correction itself
+    sn = amplitude * fmaf(rest, c, s * near_one);
+    cs = amplitude * fmaf(-rest, s, c * near_one);
 }
 
 // buf [n] float32 (one warp's): the first 2 pairs entries turned by sign * pos * freq, written to dst as T.
@@ -616,8 +617,8 @@ __global__ void __launch_bounds__(256) qkv_headnorm_rope_cache_kernel(const atom
 
 template <typename T>
 __global__ void __launch_bounds__(256) rotate_heads_kernel(T *__restrict__ x, const int64_t *__restrict__ positions,
-                                                           const float *__restrict__ freq, int H, int n, int pairs, int interleaved,
-                                                           float sign) {
+                                                           const float *__restrict__ freq, const float *__restrict__ freq_lo, float amplitude,
+                                                           int H, int n, int pairs, int interleaved, float sign) {
     pdl_launch_dependents();
     pdl_wait();
     const int64_t t = blockIdx.x;
@@ -627,7 +628,7 @@ __global__ void __launch_bounds__(256) rotate_heads_kernel(T *__restrict__ x, co
         const int h = idx / pairs, i = idx % pairs;
         const int ia = h * n + (interleaved ? 2 * i : i), ib = h * n + (interleaved ? 2 * i + 1 : i + pairs);
         float sn, cs;
-        sincosf(pos * freq[i], &sn, &cs);
+        turn(pos, freq[i], freq_lo ? freq_lo[i] : 0.f, amplitude, sn, cs);
         sn *= sign;
         const float u = to_f(row[ia]), v = to_f(row[ib]);
         row[ia] = from_f<T>(u * cs - v * sn);
@@ -866,8 +867,8 @@ bool hyb_qkv_headnorm_rope_cache(const atoma_qkv_rope_args &a, cudaStream_t stre
 #undef CALL
 }
 
-bool hyb_rotate_heads(void *x, const int64_t *positions, const float *freq, int64_t T, int64_t H, int64_t n, int64_t pairs, int32_t interleaved,
-                      float sign, uint32_t dtype, cudaStream_t stream) {
+bool hyb_rotate_heads(void *x, const int64_t *positions, const float *freq, const float *freq_lo, float amplitude, int64_t T, int64_t H, int64_t n,
+                      int64_t pairs, int32_t interleaved, float sign, uint32_t dtype, cudaStream_t stream) {
     if (T <= 0 || pairs <= 0) return true;
     if (!hybrid::known_dtype(dtype, "atoma_rotate_heads")) return false;
     if (!x || !positions || !freq || H <= 0 || 2 * pairs > n) {
@@ -875,7 +876,7 @@ bool hyb_rotate_heads(void *x, const int64_t *positions, const float *freq, int6
         return false;
     }
 #define CALL(TT) launch_ex(rotate_heads_kernel<TT>, dim3(static_cast<unsigned>(T)), dim3(256), 0, stream, static_cast<TT *>(x), positions, freq, \
-                           static_cast<int>(H), static_cast<int>(n), static_cast<int>(pairs), interleaved, sign)
+                           freq_lo, amplitude, static_cast<int>(H), static_cast<int>(n), static_cast<int>(pairs), interleaved, sign)
     return hybrid::launched(HYB_DISPATCH(dtype, CALL), "rotate_heads_kernel");
 #undef CALL
 }
@@ -974,10 +975,10 @@ extern "C" void atoma_qkv_headnorm_rope_cache(const atoma_qkv_rope_args *args, a
     hyb_qkv_headnorm_rope_cache(*args, static_cast<cudaStream_t>(stream));
 }
 
-extern "C" void atoma_rotate_heads(void *x, const int64_t *positions, const float *freq, int64_t T, int64_t H, int64_t n, int64_t pairs,
-                                   int32_t interleaved, float sign, uint32_t dtype, atoma_stream_t stream) {
+extern "C" void atoma_rotate_heads(void *x, const int64_t *positions, const float *freq, const float *freq_lo, float amplitude, int64_t T, int64_t H,
+                                   int64_t n, int64_t pairs, int32_t interleaved, float sign, uint32_t dtype, atoma_stream_t stream) {
     clear_status();
-    hyb_rotate_heads(x, positions, freq, T, H, n, pairs, interleaved, sign, dtype, static_cast<cudaStream_t>(stream));
+    hyb_rotate_heads(x, positions, freq, freq_lo, amplitude, T, H, n, pairs, interleaved, sign, dtype, static_cast<cudaStream_t>(stream));
 }
 
 extern "C" void atoma_latent_norm_rope_cache(const void *proj, int64_t ld, const float *q_weight, const float *kv_weight, const float *freq, const float *freq_lo, float amplitude,

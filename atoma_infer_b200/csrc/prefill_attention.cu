@@ -19,7 +19,13 @@
 //    exponentiated; the epilogue reads O from tensor memory, scales by 1/rowsum and stores 16-byte
 //    vectors;
 //  * tiles that stick out of their sequence (ragged tails) are loaded with cp.async + zero fill in
-//    the same swizzled layout instead of TMA, so nothing outside a sequence is ever multiplied in.
+//    the same swizzled layout instead of TMA, so nothing outside a sequence is ever multiplied in;
+//  * query / key heads may be longer than value heads (KH 64-column pieces of them, zero-filled behind their
+//    last entry): 128 columns over values of 64, 192 over values of 128 (one key stage instead of two there:
+//    two query tiles, one key and two value stages take 208 KB of shared memory);
+//  * every wait is bounded: a wait that runs out makes the CTA's roles leave their loops, the copies in
+//    flight are waited for (again with a bound), tensor memory is freed and a counter is raised that
+//    the host can read (atoma_prefill_timeouts).
 //
 // Bound: tensor pipe.  Algorithmic flops: 4 * sum_b(visible (q,k) pairs) * D per head.
 #include "common.cuh"
@@ -35,19 +41,36 @@ namespace {
 constexpr int kPfThreads = 384;  // warpgroup 0: loads (warp 0) + MMA issue (warp 1); warpgroups 1, 2: softmax
 constexpr int kPfM = 128, kPfN = 128;
 constexpr int kQTiles = 2;       // two 128-row query tiles per CTA, one softmax warpgroup each
-constexpr int kKvStages = 2;
+constexpr int kVStages = 2;
+constexpr int kPfWaitTries = 1 << 22;   // a try suspends the thread for up to a hardware-chosen time: seconds in all
 constexpr int kTmemCols = 512;   // S_A 0..127 | S_B 128..255 | O_A 256.. | O_B 384..
 constexpr int kPfIssueRegs = 56, kPfSoftmaxRegs = 224;  // setmaxnreg: 168 * 384 = 56 * 128 + 224 * 256
 constexpr float kRescaleThreshold = 8.f;  // log2 units: P <= 2^8 between corrections
 constexpr int kPfBiasSmem = 2048;         // distances whose bias (this head's column of the table) is kept in shared memory
 
-template <int D>
+__device__ unsigned int g_prefill_late;   // CTAs that gave up waiting, since the library was loaded
+
+template <int D, int KH>
 struct PfCfg {
-    static constexpr int kHalves = D / 64;
-    static constexpr int kHalfBytes = 128 * 128;            // 128 rows of 128 bytes
-    static constexpr int kTileBytes = kHalves * kHalfBytes;  // one Q / K / V tile
-    static constexpr int kSmem = kTileBytes * (kQTiles + 2 * kKvStages) + 1024;
+    static constexpr int kHalfBytes = 128 * 128;             // 128 rows of 128 bytes
+    static constexpr int kQkBytes = KH * kHalfBytes;         // one Q / K tile
+    static constexpr int kVBytes = (D / 64) * kHalfBytes;    // one V tile
+    static constexpr int kKStages = KH > 2 ? 1 : 2;
+    static constexpr int kSmem = kQkBytes * (kQTiles + kKStages) + kVBytes * kVStages + 1024;
 };
+
+// A bounded wait of a whole warp (converged; the result is the same for every lane).  `late` (shared) is raised when the bound is
+// reached and makes every other wait of the CTA give up as well.
+__device__ __forceinline__ bool pf_wait(uint64_t *bar, uint32_t parity, volatile int *late) {
+    bool ok = false;
+    for (int i = 0; i < kPfWaitTries; ++i) {
+        ok = mbar_try_wait(bar, parity);
+        if (ok || ((i & 255) == 255 && *late)) break;
+    }
+    ok = __all_sync(0xffffffffu, ok);
+    if (!ok) *late = 1;
+    return ok;
+}
 
 struct PfSeq {
     int len_q, len_k;
@@ -78,19 +101,22 @@ __device__ __forceinline__ PfSeq pf_seq(const MhaParams &p, int bidb) {
 
 // BIASED: a bias by query-key distance is added to the scaled scores (MhaParams::dist_bias); an instantiation of its own, so
 // that the unbiased kernel keeps its register allocation.
-template <typename T, int D, bool BIASED>
+template <typename T, int D, int KH, bool BIASED>
 __global__ void __launch_bounds__(kPfThreads, 1)
 prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                     const __grid_constant__ CUtensorMap map_v, const MhaParams p) {
-    using C = PfCfg<D>;
+    using C = PfCfg<D, KH>;
+    constexpr int kKStages = C::kKStages;
     extern __shared__ unsigned char smem_dyn[];
     unsigned char *tiles = smem_dyn + ((1024u - (smem_u32(smem_dyn) & 1023u)) & 1023u);
     unsigned char *sq = tiles;                            // [q tile]
-    unsigned char *sk = sq + kQTiles * C::kTileBytes;     // [stage]
-    unsigned char *sv = sk + kKvStages * C::kTileBytes;   // [stage]
-    __shared__ __align__(8) uint64_t q_full[kQTiles], k_full[kKvStages], k_empty[kKvStages], v_full[kKvStages],
-        v_empty[kKvStages], s_full[kQTiles], p_full[kQTiles], pv_done[kQTiles];
+    unsigned char *sk = sq + kQTiles * C::kQkBytes;       // [stage]
+    unsigned char *sv = sk + kKStages * C::kQkBytes;      // [stage]
+    __shared__ __align__(8) uint64_t q_full[kQTiles], k_full[kKStages], k_empty[kKStages], v_full[kVStages],
+        v_empty[kVStages], s_full[kQTiles], p_full[kQTiles], pv_done[kQTiles];
     __shared__ uint32_t tmem_base_smem;
+    __shared__ int late_s;
+    volatile int *late = &late_s;
     __shared__ float bias_s[BIASED ? kPfBiasSmem : 1];
 
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -98,9 +124,12 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
     const int head = blockIdx.y, bidb = blockIdx.z;
 
     if (tid == 0) {
-        for (int i = 0; i < kKvStages; ++i) {
+        late_s = 0;
+        for (int i = 0; i < kKStages; ++i) {
             mbar_init(&k_full[i], 1);
             mbar_init(&k_empty[i], 1);
+        }
+        for (int i = 0; i < kVStages; ++i) {
             mbar_init(&v_full[i], 1);
             mbar_init(&v_empty[i], 1);
         }
@@ -161,21 +190,23 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             // ================================ loads ================================
             // A tile that lies completely inside its sequence is one TMA transaction (kHalves boxes);
             // a ragged one is filled with cp.async + zero fill in the same 128-byte-swizzled layout.
-            auto load_tile = [&](unsigned char *dst, const CUtensorMap *map, uint64_t *bar, const T *gbase,
+            // Q and K tiles are KH pieces of 64 columns, V tiles D / 64; columns from `cols` on are zero (TMA's fill).
+            auto load_tile = [&](auto pieces, int cols, unsigned char *dst, const CUtensorMap *map, uint64_t *bar, const T *gbase,
                                  int64_t rs, int row0, int len, int tma_row, int tma_head, int tma_batch,
                                  uint64_t policy) {
+                constexpr int NP = decltype(pieces)::value;
                 if (row0 + 128 <= len) {
                     if (elect_one_sync()) {
-                        mbar_arrive_expect_tx(bar, C::kTileBytes);
+                        mbar_arrive_expect_tx(bar, NP * C::kHalfBytes);
 #pragma unroll
-                        for (int hf = 0; hf < C::kHalves; ++hf)
+                        for (int hf = 0; hf < NP; ++hf)
                             tma_load_4d(dst + hf * C::kHalfBytes, map, bar, hf * 64, tma_head, tma_row, tma_batch, policy);
                     }
                     __syncwarp();
                 } else {
-                    for (int idx = lane; idx < 128 * (D / 8); idx += 32) {
-                        const int r = idx / (D / 8), c = idx % (D / 8);
-                        const bool ok = row0 + r < len;
+                    for (int idx = lane; idx < 128 * NP * 8; idx += 32) {
+                        const int r = idx / (NP * 8), c = idx % (NP * 8);
+                        const bool ok = row0 + r < len && c * 8 < cols;
                         const T *src = ok ? gbase + static_cast<int64_t>(row0 + r) * rs + c * 8 : gbase;
                         cp_async_16(smem_u32(dst + (c >> 3) * C::kHalfBytes + r * 128 + (((c & 7) ^ (r & 7)) << 4)), src,
                                     ok ? 16 : 0);
@@ -187,23 +218,38 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     if (lane == 0) mbar_arrive(bar);
                 }
             };
+            using QkPieces = std::integral_constant<int, KH>;
+            using VPieces = std::integral_constant<int, D / 64>;
+            const int d_k = p.d_k > 0 ? p.d_k : D;
             const T *qg = static_cast<const T *>(p.q) + si.q_off + static_cast<int64_t>(head) * p.q_hs;
             const T *kg = static_cast<const T *>(p.k) + si.k_off + static_cast<int64_t>(kvh) * p.k_hs;
             const T *vg = static_cast<const T *>(p.v) + si.v_off + static_cast<int64_t>(kvh) * p.v_hs;
 #pragma unroll
             for (int t = 0; t < kQTiles; ++t)
                 if (nt[t] > 0)
-                    load_tile(sq + t * C::kTileBytes, &map_q, &q_full[t], qg, p.q_rs, m0[t], len_q, si.q_row0 + m0[t],
+                    load_tile(QkPieces(), d_k, sq + t * C::kQkBytes, &map_q, &q_full[t], qg, p.q_rs, m0[t], len_q, si.q_row0 + m0[t],
                               head, si.q_batch, kL2EvictFirst);
+            int k_issued = 0, v_issued = 0;
             for (int j = n_lo; j < n_max; ++j) {
-                const int s = (j - n_lo) % kKvStages;
-                const uint32_t par = (((j - n_lo) / kKvStages) & 1) ^ 1;
-                mbar_wait(&k_empty[s], par);
-                load_tile(sk + s * C::kTileBytes, &map_k, &k_full[s], kg, p.k_rs, j * kPfN, len_k,
+                const int jj = j - n_lo, ks = jj % kKStages, vs = jj % kVStages;
+                if (!pf_wait(&k_empty[ks], ((jj / kKStages) & 1) ^ 1, late)) break;
+                load_tile(QkPieces(), d_k, sk + ks * C::kQkBytes, &map_k, &k_full[ks], kg, p.k_rs, j * kPfN, len_k,
                           si.k_row0 + j * kPfN, kvh, si.k_batch, kL2EvictLast);
-                mbar_wait(&v_empty[s], par);
-                load_tile(sv + s * C::kTileBytes, &map_v, &v_full[s], vg, p.v_rs, j * kPfN, len_k,
+                ++k_issued;
+                if (!pf_wait(&v_empty[vs], ((jj / kVStages) & 1) ^ 1, late)) break;
+                load_tile(VPieces(), D, sv + vs * C::kVBytes, &map_v, &v_full[vs], vg, p.v_rs, j * kPfN, len_k,
                           si.k_row0 + j * kPfN, kvh, si.k_batch, kL2EvictLast);
+                ++v_issued;
+            }
+            if (v_issued < n_max - n_lo) {   // a wait ran out: the copies in flight land before the CTA goes away
+                auto landed = [&](uint64_t *bar, uint32_t parity) {
+                    for (int i = 0; i < kPfWaitTries && !mbar_try_wait(bar, parity); ++i) {
+                    }
+                };
+                for (int t = 0; t < kQTiles; ++t)
+                    if (nt[t] > 0) landed(&q_full[t], 0);
+                for (int i = max(0, k_issued - kKStages); i < k_issued; ++i) landed(&k_full[i % kKStages], (i / kKStages) & 1);
+                for (int i = max(0, v_issued - kVStages); i < v_issued; ++i) landed(&v_full[i % kVStages], (i / kVStages) & 1);
             }
         } else if (warp == 1 && n_max > 0) {
             // ================================ MMA issue ================================
@@ -218,13 +264,12 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             const uint32_t idesc_qk = umma_idesc_f16(kPfM, kPfN, kBf16, false);
             const uint32_t idesc_pv = umma_idesc_f16(kPfM, D, kBf16, true);
             auto issue_qk = [&](int t, int j) {
-                const int s = (j - n_lo) % kKvStages;
-                const uint32_t q_addr = smem_u32(sq + t * C::kTileBytes);
-                const uint32_t k_addr = smem_u32(sk + s * C::kTileBytes);
+                const uint32_t q_addr = smem_u32(sq + t * C::kQkBytes);
+                const uint32_t k_addr = smem_u32(sk + (j - n_lo) % kKStages * C::kQkBytes);
                 const uint32_t tmem_s = tmem_base + t * 128;
                 if (elect_one_sync()) {
 #pragma unroll
-                    for (int kk = 0; kk < D / 16; ++kk) {
+                    for (int kk = 0; kk < KH * 4; ++kk) {
                         const uint32_t off = (kk >> 2) * C::kHalfBytes + (kk & 3) * 32;
                         umma_f16_ss(tmem_s, umma_desc_k_sw128(q_addr + off), umma_desc_k_sw128(k_addr + off), idesc_qk,
                                     kk != 0 ? 1u : 0u);
@@ -234,8 +279,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 __syncwarp();
             };
             auto issue_pv = [&](int t, int j) {
-                const int s = (j - n_lo) % kKvStages;
-                const uint32_t v_addr = smem_u32(sv + s * C::kTileBytes);
+                const uint32_t v_addr = smem_u32(sv + (j - n_lo) % kVStages * C::kVBytes);
                 const uint32_t tmem_p = tmem_base + t * 128;
                 const uint32_t tmem_o = tmem_base + 256 + t * 128;
                 if (elect_one_sync()) {
@@ -250,36 +294,36 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 __syncwarp();
             };
             // first key tile: both query tiles
-            mbar_wait(&k_full[0], 0);
+            bool ok = pf_wait(&k_full[0], 0, late);
 #pragma unroll
             for (int t = 0; t < kQTiles; ++t) {
                 if (nt[t] > 0) {
-                    mbar_wait(&q_full[t], 0);
+                    ok = ok && pf_wait(&q_full[t], 0, late);
                     tc_fence_after_sync();
-                    issue_qk(t, n_lo);
+                    if (ok) issue_qk(t, n_lo);
                 }
             }
             if (elect_one_sync()) umma_commit(&k_empty[0]);
             __syncwarp();
-            for (int j = n_lo; j < n_max; ++j) {
+            for (int j = n_lo; ok && j < n_max; ++j) {
                 const int jj = j - n_lo;
-                const int s = jj % kKvStages, sn = (jj + 1) % kKvStages;
-                mbar_wait(&v_full[s], (jj / kKvStages) & 1);
+                const int s = jj % kVStages, sn = (jj + 1) % kKStages;
+                ok = pf_wait(&v_full[s], (jj / kVStages) & 1, late);
                 bool k_next_ready = false;
 #pragma unroll
                 for (int t = 0; t < kQTiles; ++t) {
                     if (j < nt[t]) {
-                        mbar_wait(&p_full[t], jj & 1);
+                        ok = ok && pf_wait(&p_full[t], jj & 1, late);
                         tc_fence_after_sync();
-                        issue_pv(t, j);
+                        if (ok) issue_pv(t, j);
                     }
                     if (j + 1 < nt[t]) {
                         if (!k_next_ready) {
-                            mbar_wait(&k_full[sn], ((jj + 1) / kKvStages) & 1);
+                            ok = ok && pf_wait(&k_full[sn], ((jj + 1) / kKStages) & 1, late);
                             k_next_ready = true;
                         }
                         tc_fence_after_sync();
-                        issue_qk(t, j + 1);
+                        if (ok) issue_qk(t, j + 1);
                     }
                 }
                 if (elect_one_sync()) {
@@ -315,7 +359,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 l_run = 1.f;
             }
             for (int j = n_lo; j < n_tiles; ++j) {
-                mbar_wait(&s_full[t], (j - n_lo) & 1);
+                if (!pf_wait(&s_full[t], (j - n_lo) & 1, late)) break;
                 tc_fence_after_sync();
                 uint32_t sv_[128];
 #pragma unroll
@@ -376,7 +420,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                     if (j > n_lo) {
                         // O of this row lives in tensor memory: wait until P.V of the previous tile has
                         // been accumulated, rescale, write back.  Rare after the first tiles.
-                        mbar_wait(&pv_done[t], (j - 1 - n_lo) & 1);
+                        pf_wait(&pv_done[t], (j - 1 - n_lo) & 1, late);
                         tc_fence_after_sync();
 #pragma unroll
                         for (int c = 0; c < D / 32; ++c) {
@@ -412,16 +456,27 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 if (lane == 0) mbar_arrive(&p_full[t]);
             }
             // ---- epilogue: O / rowsum -> global ----
-            mbar_wait(&pv_done[t], (n_tiles - 1 - n_lo) & 1);
+            pf_wait(&pv_done[t], (n_tiles - 1 - n_lo) & 1, late);
             tc_fence_after_sync();
             const bool empty = (l_run == 0.f || l_run != l_run);
             const float inv = empty ? 0.f : 1.f / l_run;
+            const T *gg = p.gate ? static_cast<const T *>(p.gate) + static_cast<int64_t>(si.q_row0 + grow) * p.gate_rs + static_cast<int64_t>(head) * D : nullptr;
 #pragma unroll
             for (int c = 0; c < D / 32; ++c) {
                 uint32_t ov[32];
                 tmem_ld_32x32b_x32(tmem_o + c * 32, ov);
                 tmem_ld_wait();
                 if (grow < len_q) {
+                    if (gg) {
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) {
+                            const uint4 g = *reinterpret_cast<const uint4 *>(gg + c * 32 + i * 8);
+                            const T *ge = reinterpret_cast<const T *>(&g);
+#pragma unroll
+                            for (int e = 0; e < 8; ++e)
+                                ov[8 * i + e] = __float_as_uint(__uint_as_float(ov[8 * i + e]) / (1.f + __expf(-static_cast<float>(ge[e]))));
+                        }
+                    }
 #pragma unroll
                     for (int i = 0; i < 4; ++i) {
                         uint4 w;
@@ -449,6 +504,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
         tc_fence_after_sync();
         tmem_dealloc(tmem_base, kTmemCols);
     }
+    if (tid == 0 && *late) atomicAdd(&g_prefill_late, 1u);
 }
 
 // ---------------------------------------------------------------------------------------------
@@ -494,13 +550,13 @@ bool make_attn_map(CUtensorMap *out, const void *ptr, int d, int heads, int64_t 
     return true;
 }
 
-template <typename T, int D, bool BIASED>
+template <typename T, int D, int KH, bool BIASED>
 bool launch_prefill_b(const CUtensorMap &mq, const CUtensorMap &mk, const CUtensorMap &mv, const MhaParams &p, cudaStream_t stream) {
-    constexpr size_t smem = PfCfg<D>::kSmem;
+    constexpr size_t smem = PfCfg<D, KH>::kSmem;
     static thread_local int attr_dev = -1;
     const DeviceInfo &di = current_device_info();
     if (attr_dev != di.ordinal) {
-        cudaError_t e = cudaFuncSetAttribute(prefill_attn_kernel<T, D, BIASED>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        cudaError_t e = cudaFuncSetAttribute(prefill_attn_kernel<T, D, KH, BIASED>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                              static_cast<int>(smem));
         if (e != cudaSuccess) {
             set_status(static_cast<int>(e), "prefill: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
@@ -509,7 +565,7 @@ bool launch_prefill_b(const CUtensorMap &mq, const CUtensorMap &mk, const CUtens
         attr_dev = di.ordinal;
     }
     dim3 grid((p.seqlen_q + kQTiles * kPfM - 1) / (kQTiles * kPfM), p.h, p.b);
-    prefill_attn_kernel<T, D, BIASED><<<grid, kPfThreads, smem, stream>>>(mq, mk, mv, p);
+    prefill_attn_kernel<T, D, KH, BIASED><<<grid, kPfThreads, smem, stream>>>(mq, mk, mv, p);
     note_launch();
     return check_launch("prefill_attn_kernel");
 }
@@ -517,7 +573,8 @@ bool launch_prefill_b(const CUtensorMap &mq, const CUtensorMap &mk, const CUtens
 template <typename T, int D>
 bool launch_prefill(const CUtensorMap &mq, const CUtensorMap &mk, const CUtensorMap &mv, const MhaParams &p,
                     cudaStream_t stream) {
-    return (p.dist_bias && p.dist_rows > 0) ? launch_prefill_b<T, D, true>(mq, mk, mv, p, stream) : launch_prefill_b<T, D, false>(mq, mk, mv, p, stream);
+    return (p.dist_bias && p.dist_rows > 0) ? launch_prefill_b<T, D, D / 64, true>(mq, mk, mv, p, stream)
+                                            : launch_prefill_b<T, D, D / 64, false>(mq, mk, mv, p, stream);
 }
 
 }  // namespace
@@ -529,6 +586,8 @@ int try_launch_prefill_tc(const MhaParams &p, bool is_bf16, cudaStream_t stream)
     if (p.seqlen_q < 32) return 0;  // a 128-row tile would be mostly padding
     if (!(p.scale_log2 > 0.f)) return 0;
     if (p.h_k <= 0 || p.h % p.h_k != 0 || p.h > 65535 || p.b > 65535) return 0;
+    if (p.d_k > 0 && (p.d_k % 8 || p.d_k > p.d + 64 || (p.d_k > p.d && (!is_bf16 || p.dist_bias)))) return 0;
+    if (p.gate && (!p.cu_q || p.gate_rs % 8 || (reinterpret_cast<uintptr_t>(p.gate) & 15))) return 0;
     const DeviceInfo &di = current_device_info();
     if (di.cc_major != 10) return 0;
     // TMA: 16-byte aligned bases and strides (run_mha already checked pointers and strides % 8)
@@ -548,11 +607,15 @@ int try_launch_prefill_tc(const MhaParams &p, bool is_bf16, cudaStream_t stream)
     const int64_t q_bs = (q_varlen || p.b == 1 || p.q_bs == 0) ? p.q_rs : p.q_bs;
     const int64_t k_bs = (k_varlen || p.b == 1 || p.k_bs == 0) ? p.k_rs : p.k_bs;
     const int64_t v_bs = (k_varlen || p.b == 1 || p.v_bs == 0) ? p.v_rs : p.v_bs;
-    if (!make_attn_map(&mq, p.q, p.d, p.h, q_rows, q_b, p.q_hs, p.q_rs, q_bs, is_bf16)) return -1;
-    if (!make_attn_map(&mk, p.k, p.d, p.h_k, k_rows, k_b, p.k_hs, p.k_rs, k_bs, is_bf16)) return -1;
+    const int d_k = p.d_k > 0 ? p.d_k : p.d;
+    if (!make_attn_map(&mq, p.q, d_k, p.h, q_rows, q_b, p.q_hs, p.q_rs, q_bs, is_bf16)) return -1;
+    if (!make_attn_map(&mk, p.k, d_k, p.h_k, k_rows, k_b, p.k_hs, p.k_rs, k_bs, is_bf16)) return -1;
     if (!make_attn_map(&mv, p.v, p.d, p.h_k, k_rows, k_b, p.v_hs, p.v_rs, v_bs, is_bf16)) return -1;
     bool ok;
-    if (is_bf16) ok = p.d == 128 ? launch_prefill<__nv_bfloat16, 128>(mq, mk, mv, p, stream)
+    if ((d_k + 63) / 64 > p.d / 64)   // longer query / key heads than value heads
+        ok = p.d == 128 ? launch_prefill_b<__nv_bfloat16, 128, 3, false>(mq, mk, mv, p, stream)
+                        : launch_prefill_b<__nv_bfloat16, 64, 2, false>(mq, mk, mv, p, stream);
+    else if (is_bf16) ok = p.d == 128 ? launch_prefill<__nv_bfloat16, 128>(mq, mk, mv, p, stream)
                                  : launch_prefill<__nv_bfloat16, 64>(mq, mk, mv, p, stream);
     else ok = p.d == 128 ? launch_prefill<__half, 128>(mq, mk, mv, p, stream)
                          : launch_prefill<__half, 64>(mq, mk, mv, p, stream);
@@ -560,3 +623,9 @@ int try_launch_prefill_tc(const MhaParams &p, bool is_bf16, cudaStream_t stream)
 }
 
 }  // namespace atoma
+
+extern "C" int atoma_prefill_timeouts(void) {
+    unsigned int n = 0;
+    if (cudaMemcpyFromSymbol(&n, atoma::g_prefill_late, sizeof(n)) != cudaSuccess) return -1;
+    return static_cast<int>(n);
+}

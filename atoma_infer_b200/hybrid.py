@@ -617,10 +617,10 @@ class HybridExecutor:
         def stack(rows_of, bias=None) -> int:
             at, n = sum(p.shape[0] for p in parts), sum(t.shape[0] for t in rows_of)
             parts.extend(rows_of)
-            biases.append(bias.float() if bias is not None else torch.zeros(n))
+            biases.append(bias.float().cpu() if bias is not None else torch.zeros(n))
             pad = -n % 8
             if pad:
-                parts.append(torch.zeros((pad, W), dtype=rows_of[0].dtype))
+                parts.append(torch.zeros((pad, W), dtype=rows_of[0].dtype, device=rows_of[0].device))
                 biases.append(torch.zeros(pad))
             return at
 
@@ -658,6 +658,13 @@ class HybridExecutor:
             L.w_uv = big(need("w_uv", (a.heads * a.vdim, a.kv_rank))).data_ptr()
             L.w_o = big(need("w_o", (W, a.heads * a.vdim))).data_ptr()
             L.rot_amplitude = 1.0
+            if (self.dtype == torch.bfloat16 and a.vdim in (64, 128) and a.dim + a.rot_dim <= a.vdim + 64 and
+                    all(v % 8 == 0 for v in (a.dim + a.rot_dim, a.kv_rank, a.kv_rank + a.rot_dim))):
+                # a cached row -> whole keys of all heads (long portions): a head's rows are [w_uk | 0] and [0 | identity]
+                rows = torch.zeros((a.heads, a.dim + a.rot_dim, a.kv_rank + a.rot_dim), dtype=w["w_uk"].dtype, device=w["w_uk"].device)
+                rows[:, :a.dim, :a.kv_rank] = w["w_uk"].reshape(a.heads, a.dim, a.kv_rank)
+                rows[:, a.dim:, a.kv_rank:] = torch.eye(a.rot_dim, dtype=rows.dtype, device=rows.device)
+                L.w_uk_rot = big(rows.reshape(a.heads * (a.dim + a.rot_dim), -1)).data_ptr()
             if a.rot_dim > 0:
                 self._place_rotation(L, i, a.rotary or RotarySpec(dims=a.rot_dim), a.rot_dim, small)
         elif ls.mixer == "lru":

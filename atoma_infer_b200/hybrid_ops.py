@@ -285,13 +285,14 @@ def finish_logits_greedy(logits, scale, softcap):
 
 
 def latent_attention_expanded(q, cache, w_uk, w_uv, query_start, context_lens, block_tables, sink, H, dim, R, block_size, window, scale,
-                              min_q, max_query_len, max_seq_len, max_keys, out=None):
+                              min_q, max_query_len, max_seq_len, max_keys, out=None, rot_dim=0, vdim=0, gate=None):
     """Rows of sequences with at least min_q tokens in the step are written; the others are left as they are in `out`."""
     from ._lib import LatentExpandedArgs
     T = q.shape[0]
     if out is None:
-        out = torch.zeros((T, H * dim), dtype=q.dtype, device=q.device)
+        out = torch.zeros((T, H * (vdim or dim)), dtype=q.dtype, device=q.device)
     a = LatentExpandedArgs()
+    a.rot_dim, a.vdim, a.gate, a.ld_gate = rot_dim, vdim, _p(gate), 0 if gate is None else gate.stride(0)
     a.q, a.latent_cache, a.w_uk, a.w_uv, a.out = _p(q), _p(cache), _p(w_uk), _p(w_uv), _p(out)
     a.query_start, a.context_lens, a.block_tables, a.sink = _p(query_start), _p(context_lens), _p(block_tables), _p(sink)
     a.T, a.B, a.max_blocks, a.H, a.dim, a.R = T, block_tables.shape[0], block_tables.shape[1], H, dim, R
@@ -527,9 +528,9 @@ def qkv_headnorm_rope_cache(proj, q_off, k_off, v_off, q_w, k_w, qk_freq, v_freq
     return q
 
 
-def rotate_heads(x, positions, freq, H, n, interleaved, sign):
+def rotate_heads(x, positions, freq, H, n, interleaved, sign, freq_lo=None, amplitude=1.0):
     """In place on x [T, H n]."""
-    _lib.lib().atoma_rotate_heads(_p(x), _p(positions), _p(freq), x.shape[0], H, n, freq.numel(), int(interleaved), sign, _CODES[x.dtype], _s())
+    _lib.lib().atoma_rotate_heads(_p(x), _p(positions), _p(freq), _p(freq_lo), amplitude, x.shape[0], H, n, freq.numel(), int(interleaved), sign, _CODES[x.dtype], _s())
     _check()
     return x
 
@@ -607,3 +608,8 @@ def linear_scan(decay, inp, gate, gate_bias, state, state_slots, query_start, co
     _lib.lib().atoma_linear_scan(C.byref(a), _s())
     _check()
     return out
+
+
+def prefill_timeouts() -> int:
+    """CTAs of the tensor-memory prefill attention kernel that gave up a wait since the library was loaded."""
+    return int(_lib.lib().atoma_prefill_timeouts())

@@ -234,12 +234,17 @@ typedef struct atoma_latent_attn_args {
 void atoma_latent_attention_paged(const atoma_latent_attn_args *args, atoma_stream_t stream);
 
 /*
- * The same attention for LONG prompt portions, on expanded keys and values (bfloat16, dim = vdim of 64 or 128): for every
+ * The same attention for LONG prompt portions, on expanded keys and values (bfloat16, values of 64 or 128, keys of up to 64 more
+ * entries): for every
  * sequence with at least min_q query tokens in the step, the latents its queries can see (window + portion) are gathered
  * from the paged cache, k = w_uk c and v = w_uv c are formed by two dense products, and softmax attention with the window
  * and the sink runs per head on the 5th-generation tensor cores; out[t, h dim ..] is written for those sequences' tokens
  * only.  A (query, key, head) pair costs 2 (dim + vdim) multiply-adds here instead of 4 kv_rank in the latent space.
  * max_keys: an upper bound of the gathered rows (sum over the long sequences of min(context, window - 1) + tokens).
+ * Cached rows with a score-only tail (rot_dim > 0, a rotated key part that all heads share): rows have R + rot_dim entries, query
+ * heads dim + rot_dim (their tail already rotated), and w_uk is [H (dim + rot_dim), R + rot_dim] — a head's rows [W_uk_h | 0] and
+ * [0 | identity], so that one product makes whole keys; values come from the first R entries.  gate (NULL: none, row stride ld_gate):
+ * the result times sigmoid(gate[t, h vdim + j]).
  */
 typedef struct atoma_latent_expanded_args {
     const void *q;                /* [T, H dim] */
@@ -253,6 +258,9 @@ typedef struct atoma_latent_expanded_args {
     int64_t T, B, max_blocks, H, dim, R, block_size, window, max_keys;
     float scale;
     int32_t min_q, max_query_len, max_seq_len;
+    int64_t rot_dim, vdim;        /* vdim 0: dim */
+    const void *gate;
+    int64_t ld_gate;
 } atoma_latent_expanded_args;
 void atoma_latent_attention_expanded(const atoma_latent_expanded_args *args, atoma_stream_t stream);
 
@@ -527,9 +535,10 @@ typedef struct atoma_qkv_rope_args {
 } atoma_qkv_rope_args;
 void atoma_qkv_headnorm_rope_cache(const atoma_qkv_rope_args *args, atoma_stream_t stream);
 
-/* In place on x [T, H, n] (`dtype`): the first 2 pairs entries of every head turned by sign * position * freq[i]. */
-void atoma_rotate_heads(void *x, const int64_t *positions, const float *freq, int64_t T, int64_t H, int64_t n, int64_t pairs,
-                        int32_t interleaved, float sign, uint32_t dtype, atoma_stream_t stream);
+/* In place on x [T, H, n] (`dtype`): the first 2 pairs entries of every head turned by sign * position * (freq[i] + freq_lo[i]) (freq_lo
+ * NULL: none) and scaled by `amplitude`. */
+void atoma_rotate_heads(void *x, const int64_t *positions, const float *freq, const float *freq_lo, float amplitude, int64_t T, int64_t H,
+                        int64_t n, int64_t pairs, int32_t interleaved, float sign, uint32_t dtype, atoma_stream_t stream);
 
 /*
  * Latent attention with a rotated key part.  proj[t, :] (row stride ld) = [c_q (q_rank) | c (kv_rank) | k_rot (rot_dim)]:
@@ -801,6 +810,10 @@ void atoma_hybrid_step(const atoma_hybrid_model *model, const atoma_hybrid_batch
  * bit 4 = the matrix-state scans with many rows per lane whatever the step's size (they normally take 8 rows per lane when a
  * step has few CTAs; both add in the same order). */
 void atoma_debug_hybrid(int flags);
+
+/* CTAs of the tensor-memory prefill attention kernel that gave up a wait since the library was loaded (0 unless something is broken;
+ * -1: the device could not be asked).  Synchronises the device. */
+int atoma_prefill_timeouts(void);
 
 #ifdef __cplusplus
 }

@@ -270,7 +270,7 @@ def random_weights(cfg, g):
     W, P = cfg["width"], {}
 
     def rnd(*shape, scale=1.0, shift=0.0):
-        return ((torch.randn(*shape, generator=g) * scale + shift).to(torch.bfloat16)).float()
+        return ((torch.randn(shape, generator=g) * scale + shift).to(torch.bfloat16)).float()
 
     def lin(out, inp, gain=1.0):
         return rnd(out, inp, scale=gain * inp ** -0.5)
