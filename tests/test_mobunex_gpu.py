@@ -305,8 +305,8 @@ def test_grouped_attention_on_a_mixed_batch(dtype, H, G, D, V, window):
 # ------------------------------------------------------------------------------------------------
 # latent attention
 # ------------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("dims,base,scaling", [(32, 20000.0, dict(factor=8.0, original=1024, fast=32.0, slow=1.0)), (8, 500.0, dict(factor=3.0, original=64, fast=4.0, slow=2.0)),
-                                               (64, 1e6, dict(factor=40.0, original=4096, fast=32.0, slow=1.0)), (2, 100.0, dict(factor=2.0, original=16, fast=1.0, slow=1.0)),
+@pytest.mark.parametrize("dims,base,scaling", [(24, 30000.0, dict(factor=6.0, original=2048, fast=24.0, slow=1.5)), (8, 500.0, dict(factor=3.0, original=64, fast=4.0, slow=2.0)),
+                                               (64, 1e6, dict(factor=40.0, original=4096, fast=30.0, slow=1.0)), (2, 100.0, dict(factor=2.0, original=16, fast=1.0, slow=1.0)),
                                                (16, 10000.0, None)])
 def test_yarn_frequencies_and_exact_angles(dims, base, scaling):
     """The description's frequencies against the plain rule, and a rotation at position 300 000 that float32 angles would miss by 1e-2."""
@@ -335,7 +335,7 @@ def latent_case(g, H, D, Rd, V, Rq, Rk, W, scaling=True):
 
 
 @pytest.mark.parametrize("dtype", BOTH)
-@pytest.mark.parametrize("H,D,Rd,V,Rq,Rk,window", [(3, 16, 8, 16, 24, 32, 7), (6, 64, 32, 64, 72, 128, 20), (2, 10, 6, 12, 9, 14, 0), (4, 32, 64, 48, 40, 128, 33),
+@pytest.mark.parametrize("H,D,Rd,V,Rq,Rk,window", [(3, 16, 8, 16, 24, 32, 7), (7, 64, 64, 32, 72, 192, 20), (2, 10, 6, 12, 9, 14, 0), (4, 32, 64, 48, 40, 128, 33),
                                                   (5, 16, 64, 16, 24, 192, 11)])
 def test_latent_attention_on_a_mixed_batch(dtype, H, D, Rd, V, Rq, Rk, window):
     ops = _ops()
@@ -376,7 +376,7 @@ def test_latent_attention_on_a_mixed_batch(dtype, H, D, Rd, V, Rq, Rk, window):
         at += want.shape[0]
 
 
-@pytest.mark.parametrize("H,D,Rd,V,Rk,window", [(4, 64, 32, 64, 128, 100), (2, 128, 64, 128, 192, 0), (3, 128, 64, 128, 512, 150), (2, 48, 16, 64, 64, 33),
+@pytest.mark.parametrize("H,D,Rd,V,Rk,window", [(4, 64, 24, 64, 96, 100), (2, 128, 64, 128, 192, 0), (3, 128, 64, 128, 512, 150), (2, 48, 16, 64, 64, 33),
                                                 (2, 96, 32, 128, 64, 300), (2, 64, 64, 64, 64, 1), (1, 128, 56, 128, 72, 129)])
 def test_long_portions_on_whole_keys(H, D, Rd, V, Rk, window):
     """Sequences with at least 128 tokens in the step: cached rows gathered from the pages, whole keys (plain and rotated part) and values
@@ -498,7 +498,7 @@ VARIANTS = {
                         latent=dict(heads=1, mask=dict(size=2)), rglru=dict(width=24, blocks=1, conv=1), router=dict(experts=4, top=1, groups=dict(count=4, keep=2))),
     "heads_of_64": dict(width=64, kinds=("attention", "latent_attention", "rglru"),
                         attention=dict(heads=4, kv_heads=1, dim=64, vdim=64, scale=0.125, mask=dict(size=50)),
-                        latent=dict(heads=2, dim=64, rot_dim=32, vdim=64, q_rank=48, kv_rank=96, scale=0.1, mask=dict(size=200)),
+                        latent=dict(heads=2, dim=64, rot_dim=40, vdim=64, q_rank=48, kv_rank=96, scale=0.1, mask=dict(size=200)),
                         rglru=dict(width=128, blocks=2, conv=2)),
     "heads_of_128": dict(width=64, kinds=("latent_attention", "attention"), mlps=("dense", "dense"),
                          attention=dict(heads=2, kv_heads=2, dim=128, vdim=128, scale=0.09, mask=dict(size=300)),

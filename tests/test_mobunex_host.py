@@ -91,7 +91,7 @@ def test_what_the_design_does_not_have_is_refused():
             mobunex.spec_from_config(other)
 
 
-@pytest.mark.parametrize("dims,base,scaling", [(32, 20000.0, (8.0, 1024, 32.0, 1.0)), (16, 100.0, (4.0, 64, 4.0, 0.5)), (8, 1e6, (2.0, 8, 1.0, 1.0))])
+@pytest.mark.parametrize("dims,base,scaling", [(24, 30000.0, (6.0, 2048, 24.0, 1.5)), (16, 100.0, (4.0, 64, 4.0, 0.5)), (8, 1e6, (2.0, 8, 1.0, 1.0))])
 def test_yarn_rule(dims, base, scaling):
     """Fast pairs keep their frequency, slow pairs have it divided, the share in between grows with the index."""
     r = RotarySpec(dims=dims, base=base, interleaved=True, yarn=scaling)
