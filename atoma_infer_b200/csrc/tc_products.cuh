@@ -217,28 +217,45 @@ __global__ void __launch_bounds__(128) gemm_kernel(const GemmArgs p) {
                 const int pair = p.row_pair[m];
                 ow = pair >= 0 ? p.out_weight[pair] : 0.f;
             }
+            if constexpr (EPI == kEpiLru) {
+                const TA *u = A + static_cast<int64_t>(m) * p.lda;
+                float *d_row = p.decay + static_cast<int64_t>(m) * p.ld_state + z * p.N, *x_row = p.input + static_cast<int64_t>(m) * p.ld_state + z * p.N;
+                const bool pair_store = ((p.N | p.ld_state) & 1) == 0;     // two neighbouring channels in one 8-byte store
 #pragma unroll
-            for (int ni = 0; ni < 4; ++ni)
+                for (int ni = 0; ni < 4; ++ni) {
+                    const int n = n0 + wn * 32 + ni * 8 + 2 * t4;
+                    float d[2] = {0.f, 0.f}, x[2] = {0.f, 0.f};
 #pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const int n = n0 + wn * 32 + ni * 8 + 2 * t4 + e;
-                    if (n >= p.N) continue;
-                    float v = acc[mi][ni][half * 2 + e];
-                    if constexpr (EPI == kEpiLru) {
-                        const int64_t c = z * p.N + n;
-                        float d, in;
-                        lru_gates(v + p.bias_r[c], acu[mi][ni][half * 2 + e] + p.bias_i[c], p.rate[c], hybrid::to_f(A[static_cast<int64_t>(m) * p.lda + n]), d, in);
-                        p.decay[static_cast<int64_t>(m) * p.ld_state + c] = d;
-                        p.input[static_cast<int64_t>(m) * p.ld_state + c] = in;
-                        continue;
+                    for (int e = 0; e < 2; ++e) {
+                        const int64_t c = z * p.N + n + e;
+                        if (n + e < p.N)
+                            lru_gates(acc[mi][ni][half * 2 + e] + p.bias_r[c], acu[mi][ni][half * 2 + e] + p.bias_i[c], p.rate[c], hybrid::to_f(u[n + e]), d[e], x[e]);
                     }
-                    if constexpr (EPI == kEpiGlu) v = hybrid::glu_clamped(v, acu[mi][ni][half * 2 + e], p.limit, p.alpha, p.shift);
-                    else {
-                        v *= ow;
-                        if (p.gate) v *= hybrid::sigmoidf_(hybrid::to_f(p.gate[static_cast<int64_t>(m) * p.ld_gate + z * p.o_zs + n]));
+                    if (pair_store && n + 1 < p.N) {
+                        *reinterpret_cast<float2 *>(d_row + n) = make_float2(d[0], d[1]);
+                        *reinterpret_cast<float2 *>(x_row + n) = make_float2(x[0], x[1]);
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 2; ++e)
+                            if (n + e < p.N) d_row[n + e] = d[e], x_row[n + e] = x[e];
                     }
-                    O[static_cast<int64_t>(m) * p.ldo + n] = hybrid::from_f<TO>(v);
                 }
+            } else {
+#pragma unroll
+                for (int ni = 0; ni < 4; ++ni)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e) {
+                        const int n = n0 + wn * 32 + ni * 8 + 2 * t4 + e;
+                        if (n >= p.N) continue;
+                        float v = acc[mi][ni][half * 2 + e];
+                        if constexpr (EPI == kEpiGlu) v = hybrid::glu_clamped(v, acu[mi][ni][half * 2 + e], p.limit, p.alpha, p.shift);
+                        else {
+                            v *= ow;
+                            if (p.gate) v *= hybrid::sigmoidf_(hybrid::to_f(p.gate[static_cast<int64_t>(m) * p.ld_gate + z * p.o_zs + n]));
+                        }
+                        O[static_cast<int64_t>(m) * p.ldo + n] = hybrid::from_f<TO>(v);
+                    }
+            }
         }
 }
 
