@@ -23,9 +23,9 @@
 //  * query / key heads may be longer than value heads (KH 64-column pieces of them, zero-filled behind their
 //    last entry): 128 columns over values of 64, 192 over values of 128 (one key stage instead of two there:
 //    two query tiles, one key and two value stages take 208 KB of shared memory);
-//  * every wait is bounded: a wait that runs out makes the CTA's roles leave their loops, the copies in
-//    flight are waited for (again with a bound), tensor memory is freed and a counter is raised that
-//    the host can read (atoma_prefill_timeouts).
+//  * every wait is bounded: a wait that runs out stops the CTA's loads and lets its other roles run through,
+//    its copies in flight are waited for (again with a bound), tensor memory is freed and a counter is
+//    raised that the host can read (atoma_prefill_timeouts); the CTA's outputs mean nothing then.
 //
 // Bound: tensor pipe.  Algorithmic flops: 4 * sum_b(visible (q,k) pairs) * D per head.
 #include "common.cuh"
@@ -42,7 +42,7 @@ constexpr int kPfThreads = 384;  // warpgroup 0: loads (warp 0) + MMA issue (war
 constexpr int kPfM = 128, kPfN = 128;
 constexpr int kQTiles = 2;       // two 128-row query tiles per CTA, one softmax warpgroup each
 constexpr int kVStages = 2;
-constexpr int kPfWaitTries = 1 << 22;   // a try suspends the thread for up to a hardware-chosen time: seconds in all
+constexpr int kPfWaitTries = 1 << 18;   // milliseconds at least (a try may also suspend the thread for a hardware-chosen time)
 constexpr int kTmemCols = 512;   // S_A 0..127 | S_B 128..255 | O_A 256.. | O_B 384..
 constexpr int kPfIssueRegs = 56, kPfSoftmaxRegs = 224;  // setmaxnreg: 168 * 384 = 56 * 128 + 224 * 256
 constexpr float kRescaleThreshold = 8.f;  // log2 units: P <= 2^8 between corrections
@@ -59,17 +59,21 @@ struct PfCfg {
     static constexpr int kSmem = kQkBytes * (kQTiles + kKStages) + kVBytes * kVStages + 1024;
 };
 
-// A bounded wait of a whole warp (converged; the result is the same for every lane).  `late` (shared) is raised when the bound is
-// reached and makes every other wait of the CTA give up as well.
-__device__ __forceinline__ bool pf_wait(uint64_t *bar, uint32_t parity, volatile int *late) {
-    bool ok = false;
-    for (int i = 0; i < kPfWaitTries; ++i) {
-        ok = mbar_try_wait(bar, parity);
-        if (ok || ((i & 255) == 255 && *late)) break;
-    }
-    ok = __all_sync(0xffffffffu, ok);
-    if (!ok) *late = 1;
-    return ok;
+// A bounded wait; `late` (shared) is raised when the bound is reached.  The MMA and softmax warps then run on through their loops on
+// whatever is in shared and tensor memory (every access stays in bounds, every arrival they owe is made); only the loads stop
+// (pf_wait_all).
+__device__ __forceinline__ void pf_wait(uint64_t *bar, uint32_t parity, volatile int *late) {
+#pragma unroll 1
+    for (int i = 0; !mbar_try_wait(bar, parity);)
+        if (++i == kPfWaitTries) {
+            *late = 1;
+            break;
+        }
+}
+// The same for a whole (converged) warp, with one answer for all lanes: false when the wait, or any other wait of the CTA, ran out.
+__device__ __forceinline__ bool pf_wait_all(uint64_t *bar, uint32_t parity, volatile int *late) {
+    pf_wait(bar, parity, late);
+    return !__any_sync(0xffffffffu, *late != 0);
 }
 
 struct PfSeq {
@@ -232,25 +236,24 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             int k_issued = 0, v_issued = 0;
             for (int j = n_lo; j < n_max; ++j) {
                 const int jj = j - n_lo, ks = jj % kKStages, vs = jj % kVStages;
-                if (!pf_wait(&k_empty[ks], ((jj / kKStages) & 1) ^ 1, late)) break;
+                if (!pf_wait_all(&k_empty[ks], ((jj / kKStages) & 1) ^ 1, late)) break;
                 load_tile(QkPieces(), d_k, sk + ks * C::kQkBytes, &map_k, &k_full[ks], kg, p.k_rs, j * kPfN, len_k,
                           si.k_row0 + j * kPfN, kvh, si.k_batch, kL2EvictLast);
                 ++k_issued;
-                if (!pf_wait(&v_empty[vs], ((jj / kVStages) & 1) ^ 1, late)) break;
+                if (!pf_wait_all(&v_empty[vs], ((jj / kVStages) & 1) ^ 1, late)) break;
                 load_tile(VPieces(), D, sv + vs * C::kVBytes, &map_v, &v_full[vs], vg, p.v_rs, j * kPfN, len_k,
                           si.k_row0 + j * kPfN, kvh, si.k_batch, kL2EvictLast);
                 ++v_issued;
             }
-            if (v_issued < n_max - n_lo) {   // a wait ran out: the copies in flight land before the CTA goes away
-                auto landed = [&](uint64_t *bar, uint32_t parity) {
-                    for (int i = 0; i < kPfWaitTries && !mbar_try_wait(bar, parity); ++i) {
-                    }
-                };
-                for (int t = 0; t < kQTiles; ++t)
-                    if (nt[t] > 0) landed(&q_full[t], 0);
-                for (int i = max(0, k_issued - kKStages); i < k_issued; ++i) landed(&k_full[i % kKStages], (i / kKStages) & 1);
-                for (int i = max(0, v_issued - kVStages); i < v_issued; ++i) landed(&v_full[i % kVStages], (i / kVStages) & 1);
-            }
+            // whatever happens to the other roles, the copies have landed before this warp leaves
+            auto landed = [&](uint64_t *bar, uint32_t parity) {
+                for (int i = 0; i < kPfWaitTries && !mbar_try_wait(bar, parity); ++i) {
+                }
+            };
+            for (int t = 0; t < kQTiles; ++t)
+                if (nt[t] > 0) landed(&q_full[t], 0);
+            for (int i = max(0, k_issued - kKStages); i < k_issued; ++i) landed(&k_full[i % kKStages], (i / kKStages) & 1);
+            for (int i = max(0, v_issued - kVStages); i < v_issued; ++i) landed(&v_full[i % kVStages], (i / kVStages) & 1);
         } else if (warp == 1 && n_max > 0) {
             // ================================ MMA issue ================================
             // The whole warp runs this role converged on warp-uniform values; only the tcgen05
@@ -294,36 +297,36 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 __syncwarp();
             };
             // first key tile: both query tiles
-            bool ok = pf_wait(&k_full[0], 0, late);
+            pf_wait(&k_full[0], 0, late);
 #pragma unroll
             for (int t = 0; t < kQTiles; ++t) {
                 if (nt[t] > 0) {
-                    ok = ok && pf_wait(&q_full[t], 0, late);
+                    pf_wait(&q_full[t], 0, late);
                     tc_fence_after_sync();
-                    if (ok) issue_qk(t, n_lo);
+                    issue_qk(t, n_lo);
                 }
             }
             if (elect_one_sync()) umma_commit(&k_empty[0]);
             __syncwarp();
-            for (int j = n_lo; ok && j < n_max; ++j) {
+            for (int j = n_lo; j < n_max; ++j) {
                 const int jj = j - n_lo;
                 const int s = jj % kVStages, sn = (jj + 1) % kKStages;
-                ok = pf_wait(&v_full[s], (jj / kVStages) & 1, late);
+                pf_wait(&v_full[s], (jj / kVStages) & 1, late);
                 bool k_next_ready = false;
 #pragma unroll
                 for (int t = 0; t < kQTiles; ++t) {
                     if (j < nt[t]) {
-                        ok = ok && pf_wait(&p_full[t], jj & 1, late);
+                        pf_wait(&p_full[t], jj & 1, late);
                         tc_fence_after_sync();
-                        if (ok) issue_pv(t, j);
+                        issue_pv(t, j);
                     }
                     if (j + 1 < nt[t]) {
                         if (!k_next_ready) {
-                            ok = ok && pf_wait(&k_full[sn], ((jj + 1) / kKStages) & 1, late);
+                            pf_wait(&k_full[sn], ((jj + 1) / kKStages) & 1, late);
                             k_next_ready = true;
                         }
                         tc_fence_after_sync();
-                        if (ok) issue_qk(t, j + 1);
+                        issue_qk(t, j + 1);
                     }
                 }
                 if (elect_one_sync()) {
@@ -359,7 +362,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 l_run = 1.f;
             }
             for (int j = n_lo; j < n_tiles; ++j) {
-                if (!pf_wait(&s_full[t], (j - n_lo) & 1, late)) break;
+                pf_wait(&s_full[t], (j - n_lo) & 1, late);
                 tc_fence_after_sync();
                 uint32_t sv_[128];
 #pragma unroll
