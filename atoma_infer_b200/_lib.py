@@ -201,7 +201,10 @@ class HybridLayer(C.Structure):
                 # post-norm blocks: depth average, per-head score factors, rotation details, real-gated linear recurrent unit
                 [(n, C.c_void_p) for n in ("depth_w", "q_head_scale", "qk_freq_lo")] + [("rot_amplitude", C.c_float), ("route_group_top", C.c_int32)] +
                 [(n, C.c_int64) for n in ("lru_width", "lru_blocks")] +
-                [(n, C.c_void_p) for n in ("lru_w", "lru_bias_r", "lru_bias_i", "lru_rate", "r_tap_bias", "w_uk_rot")])
+                [(n, C.c_void_p) for n in ("lru_w", "lru_bias_r", "lru_bias_i", "lru_rate", "r_tap_bias", "w_uk_rot")] +
+                # differential attention, shared caches, the sum of softmax attention and a state-space recurrence
+                [("b_o", C.c_void_p), ("v_share", C.c_int64), ("diff_lambda", C.c_float), ("diff_gain", C.c_float), ("r_skip", C.c_void_p)] +
+                [(n, C.c_int64) for n in ("r_norm_groups", "mix_cols", "r_mix_off")] + [("mix_scale", C.c_float)])
 
 
 class HybridModel(C.Structure):
@@ -213,7 +216,9 @@ class HybridModel(C.Structure):
                 [("layers", C.POINTER(HybridLayer))] +
                 [("block_style", C.c_int32), ("norm_groups", C.c_int32), ("pos_table", C.c_void_p), ("max_positions", C.c_int64),
                  ("logit_softcap", C.c_float), ("side_table", C.c_void_p), ("side_dim", C.c_int64), ("side_table_width", C.c_int64),
-                 ("lanes", C.c_int32), ("embed_scale", C.c_float), ("embed_norm", C.c_void_p), ("residual_alpha", C.c_float)])
+                 ("lanes", C.c_int32), ("embed_scale", C.c_float), ("embed_norm", C.c_void_p), ("residual_alpha", C.c_float),
+                 ("branch_scale", C.c_float), ("norm_branch", C.c_int32), ("pair_table", C.c_void_p)] +
+                [(n, C.c_int64) for n in ("pair_buckets", "pair_mul_prev", "pair_mul_cur")])
 
 
 class GatedResidualArgs(C.Structure):
@@ -244,7 +249,7 @@ class SoftmaxAttnArgs(C.Structure):
                 [(n, C.c_int64) for n in ("T", "B", "max_blocks", "H", "G", "dim", "vdim", "block_size", "window", "keep_first")] +
                 [("scale", C.c_float), ("dtype", C.c_uint32), ("max_query_len", C.c_int32), ("max_seq_len", C.c_int32),
                  ("skip_min_q", C.c_int32), ("long_min_q", C.c_int32), ("long_seqs", C.c_int32), ("long_tokens", C.c_int64),
-                 ("long_ctx_sum", C.c_int64)])
+                 ("long_ctx_sum", C.c_int64), ("ld_out", C.c_int64), ("v_share", C.c_int64)])
 
 
 class ParallelResidualArgs(C.Structure):
@@ -274,7 +279,7 @@ class StateScanArgs(C.Structure):
                 [(n, C.c_float) for n in ("tau", "q_scale", "unit_eps")] +
                 [("state", C.c_void_p), ("state_stride", C.c_int64)] +
                 [(n, C.c_void_p) for n in ("state_slots", "query_start", "context_lens", "out")] +
-                [(n, C.c_int64) for n in ("T", "B", "H", "G", "dim", "vdim")] + [("dtype", C.c_uint32)])
+                [(n, C.c_int64) for n in ("T", "B", "H", "G", "dim", "vdim")] + [("dtype", C.c_uint32), ("skip", C.c_void_p)])
 
 
 class QkvRopeArgs(C.Structure):
@@ -285,7 +290,8 @@ class QkvRopeArgs(C.Structure):
                 [("rot_pairs", C.c_int64), ("v_pairs", C.c_int64), ("interleaved", C.c_int32)] +
                 [(n, C.c_void_p) for n in ("positions", "slot_mapping", "q_out", "k_cache", "v_cache")] +
                 [(n, C.c_int64) for n in ("T", "H", "G", "dim", "vdim")] + [("eps", C.c_float), ("dtype", C.c_uint32), ("bias", C.c_void_p),
-                                                                          ("q_head_scale", C.c_void_p), ("unit_norm", C.c_int32)])
+                                                                          ("q_head_scale", C.c_void_p), ("unit_norm", C.c_int32),
+                                                                          ("qk_freq_lo", C.c_void_p), ("qk_amplitude", C.c_float), ("v_heads", C.c_int64)])
 
 
 class PostnormArgs(C.Structure):
@@ -293,7 +299,8 @@ class PostnormArgs(C.Structure):
 
     _fields_ = ([(n, C.c_void_p) for n in ("y", "expert_out", "pair_row", "top_expert")] + [("top", C.c_int64)] +
                 [(n, C.c_void_p) for n in ("x", "w_norm", "depth", "depth_w")] + [("depth_n", C.c_int64), ("h", C.c_void_p), ("trace", C.c_void_p)] +
-                [("T", C.c_int64), ("width", C.c_int64), ("alpha", C.c_float), ("eps", C.c_float), ("weight_offset", C.c_float), ("dtype", C.c_uint32)])
+                [("T", C.c_int64), ("width", C.c_int64), ("alpha", C.c_float), ("eps", C.c_float), ("weight_offset", C.c_float), ("dtype", C.c_uint32),
+                 ("norm_branch", C.c_int32), ("y_bias", C.c_void_p), ("y_scale", C.c_float), ("branch_scale", C.c_float)])
 
 
 class LruGatesArgs(C.Structure):
@@ -347,7 +354,8 @@ class HybridBatch(C.Structure):
                                            "block_tables", "state_slots", "selected", "scratch")] +
                 [("scratch_bytes", C.c_int64)] +
                 [(n, C.c_void_p) for n in ("logits", "next_tokens", "residual_trace")] +
-                [("long_seqs", C.c_int32), ("long_min_q", C.c_int32), ("long_tokens", C.c_int64), ("long_ctx_sum", C.c_int64)])
+                [("long_seqs", C.c_int32), ("long_min_q", C.c_int32), ("long_tokens", C.c_int64), ("long_ctx_sum", C.c_int64),
+                 ("prev_tokens", C.c_void_p)])
 
 
 # Exact C parameter lists, in header order.
@@ -490,6 +498,9 @@ SIGNATURES = {
     "atoma_latent_query_absorb_rope": (None, [C.c_void_p] * 4 + [C.c_float, C.c_int64, C.c_int32, C.c_void_p, C.c_void_p] + [C.c_int64] * 5 +
                                        [C.c_uint32, C.c_void_p]),
     "atoma_latent_expand_values": (None, [C.c_void_p] * 3 + [C.c_int64, C.c_void_p] + [C.c_int64] * 5 + [C.c_uint32, C.c_void_p]),
+    "atoma_differential_combine": (None, [C.c_void_p] * 2 + [C.c_int64] * 4 + [C.c_float] * 3 + [C.c_uint32, C.c_void_p]),
+    "atoma_gate_groupnorm": (None, [C.c_void_p] * 2 + [C.c_int64] + [C.c_void_p] * 2 + [C.c_int64] * 6 + [C.c_float, C.c_uint32, C.c_void_p]),
+    "atoma_embed_pairs": (None, [C.c_void_p] * 6 + [C.c_int64] * 3 + [C.c_void_p] * 2 + [C.c_int64] * 3 + [C.c_uint32, C.c_void_p]),
     "atoma_postnorm_residual": (None, [C.POINTER(PostnormArgs), C.c_void_p]),
     "atoma_lru_gates": (None, [C.POINTER(LruGatesArgs), C.c_void_p]),
     "atoma_linear_scan": (None, [C.POINTER(LinearScanArgs), C.c_void_p]),

@@ -75,6 +75,11 @@ bool hyb_postnorm_residual(const atoma_postnorm_args &, cudaStream_t);
 bool hyb_lru_gates(const atoma_lru_gates_args &, cudaStream_t);
 bool hyb_linear_scan(const atoma_linear_scan_args &, cudaStream_t);
 bool hyb_latent_expand_values(const float *, const void *, const void *, int64_t, void *, int64_t, int64_t, int64_t, int64_t, int64_t, uint32_t, cudaStream_t);
+bool hyb_embed_pairs(const uint32_t *, const int32_t *, const int32_t *, const int32_t *, const void *, const void *, int64_t, int64_t, int64_t, float *,
+                     void *, int64_t, int64_t, int64_t, uint32_t, cudaStream_t);
+bool hyb_differential_combine(const void *, void *, int64_t, int64_t, int64_t, int64_t, float, float, float, uint32_t, cudaStream_t);
+bool hyb_gate_groupnorm(const float *, const void *, int64_t, const float *, void *, int64_t, int64_t, int64_t, int64_t, int64_t, int64_t, float, uint32_t,
+                        cudaStream_t);
 int64_t hyb_moe_workspace_bytes(int64_t, int64_t, int64_t, int64_t, int64_t, uint32_t);
 bool hyb_moe_experts(const atoma_moe_args &, const void **, const int32_t **, cudaStream_t);
 
@@ -90,6 +95,7 @@ struct Widths {
     bool parallel = false, keep_embedding = false;
     int64_t lru = 0;                    // post-norm blocks: channels of a linear recurrent unit
     int64_t depth = 0;                  // float32 [T, width] planes of the average over depth
+    int64_t maps = 0;                   // output row of both maps of a differential attention
 };
 
 inline bool gated(const float *bias) { return bias != nullptr; }
@@ -109,6 +115,12 @@ Widths widths(const atoma_hybrid_model &m, int64_t T) {
             if (l.mixer == ATOMA_MIXER_SOFTMAX_ATTENTION) {
                 w.q = std::max(w.q, l.heads * l.dim);
                 w.act = std::max(w.act, l.heads * l.vdim);
+                if (l.diff_gain != 0.f) w.maps = std::max(w.maps, l.heads * l.vdim);
+            } else if (l.mixer == ATOMA_MIXER_ATTENTION_SSM) {
+                w.q = std::max(w.q, l.heads * l.dim);
+                w.act = std::max(w.act, l.mix_cols);
+                w.conv = std::max(w.conv, l.r_heads * l.r_vdim + 2 * l.r_kv_heads * l.r_dim);
+                w.of32 = std::max(w.of32, l.r_heads * l.r_vdim);
             } else if (l.mixer == ATOMA_MIXER_LATENT_ATTENTION) {
                 w.q = std::max(w.q, l.heads * (l.dim + l.rot_dim));
                 w.cq = std::max(w.cq, l.q_rank);
@@ -215,6 +227,7 @@ struct Scratch {
     char *h1, *h2, *y2, *yf, *conv;
     // post-norm blocks
     float *depth, *decay, *input;
+    char *maps;
     int64_t total;
 };
 
@@ -258,6 +271,7 @@ Scratch carve(const atoma_hybrid_model &m, int64_t T, int64_t S, void *base) {
     s.depth = reinterpret_cast<float *>(take(w.depth * T * m.width * 4));
     s.decay = reinterpret_cast<float *>(take(T * w.lru * 4));
     s.input = reinterpret_cast<float *>(take(T * w.lru * 4));
+    s.maps = take(T * w.maps * es);
     s.total = off;
     return s;
 }
@@ -816,7 +830,8 @@ bool parallel_layer(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, co
     return hyb_parallel_residual_norm(r, stream);
 }
 
-// Softmax attention of a post-norm layer: stacked projection -> biases, unit norms, per-head factor, cache write -> attention -> s.act.
+// Softmax attention of a post-norm layer: stacked projection -> biases, norms, per-head factor, rotation, cache write -> attention (two maps
+// combined when differential) -> s.act.
 bool postnorm_softmax(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, const atoma_hybrid_layer &l, const Scratch &s,
                       cudaStream_t stream) {
     atoma_qkv_rope_args q{};
@@ -826,7 +841,15 @@ bool postnorm_softmax(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, 
     q.k_off = l.k_off;
     q.v_off = l.v_off;
     q.positions = b.positions;
-    q.slot_mapping = b.slot_mapping;
+    q.slot_mapping = l.v_off >= 0 ? b.slot_mapping : nullptr;   // without projections of its own the layer reads an earlier layer's caches
+    q.q_weight = l.q_norm;
+    q.k_weight = l.k_norm;
+    q.qk_freq = l.qk_freq;
+    q.qk_freq_lo = l.qk_freq_lo;
+    q.qk_amplitude = l.rot_amplitude;
+    q.rot_pairs = l.rot_pairs;
+    q.interleaved = l.rot_interleaved;
+    q.v_heads = l.v_share > 1 ? l.kv_heads / l.v_share : 0;
     q.q_out = s.q;
     q.k_cache = l.k_cache;
     q.v_cache = l.v_cache;
@@ -841,11 +864,14 @@ bool postnorm_softmax(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, 
     q.q_head_scale = l.q_head_scale;
     q.unit_norm = 1;
     if (!hyb_qkv_headnorm_rope_cache(q, stream)) return false;
+    const bool maps = l.diff_gain != 0.f;
     atoma_softmax_attn_args a{};
     a.q = s.q;
     a.k_cache = l.k_cache;
     a.v_cache = l.v_cache;
-    a.out = s.act;
+    a.out = maps ? s.maps : s.act;
+    a.ld_out = l.mixer == ATOMA_MIXER_ATTENTION_SSM ? l.mix_cols : 0;
+    a.v_share = l.v_share;
     a.positions = b.positions;
     a.token_seq = b.token_seq;
     a.query_start = b.query_start;
@@ -867,7 +893,69 @@ bool postnorm_softmax(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, 
     a.long_seqs = b.long_seqs;
     a.long_tokens = b.long_tokens;
     a.long_ctx_sum = b.long_ctx_sum;
-    return hyb_softmax_attention(a, stream);
+    if (!hyb_softmax_attention(a, stream)) return false;
+    return !maps || hyb_differential_combine(s.maps, s.act, b.num_tokens, l.heads / 2, l.kv_heads / 2, l.vdim, l.diff_lambda, l.diff_gain, m.eps, m.dtype,
+                                             stream);
+}
+
+// State-space recurrence beside the attention of a summed layer: short filter -> scan -> gate, grouped norm -> its columns of s.act.
+bool postnorm_ssm(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, const atoma_hybrid_layer &l, const Scratch &s, cudaStream_t stream) {
+    const uint32_t dt = m.dtype;
+    const int64_t es = dt == ATOMA_DTYPE_F32 ? 4 : 2;
+    const int64_t H = l.r_heads, G = l.r_kv_heads, N = l.r_dim, V = l.r_vdim, inner = H * V, C = inner + 2 * G * N, P = l.proj_cols;
+    if (!l.layer_state) {
+        set_status(kErrInvalidArg, "atoma_hybrid_step: a recurrent layer has no state");
+        return false;
+    }
+    const int64_t hist = l.r_taps > 1 ? (l.r_taps - 1) * C : 0;
+    atoma_tap_filter_args f{};
+    f.in = s.proj + l.rv_off * es;      // [x | B | C], neighbours in the stacked projection
+    f.ld_in = P;
+    f.w1 = l.r_tap_w;
+    f.bias1 = l.r_tap_bias;
+    f.out1 = s.conv;
+    f.ld_out = C;
+    f.history = l.layer_state;
+    f.history_stride = l.layer_state_stride;
+    f.state_slots = b.state_slots;
+    f.token_seq = b.token_seq;
+    f.query_start = b.query_start;
+    f.context_lens = b.context_lens;
+    f.T = b.num_tokens;
+    f.B = b.num_seqs;
+    f.channels = C;
+    f.taps = l.r_taps;
+    f.act = 1;
+    f.dtype = dt;
+    if (!hyb_tap_filter(f, stream)) return false;
+    atoma_state_scan_args d{};
+    d.kind = 2;
+    d.v = s.conv;
+    d.k = s.conv + inner * es;
+    d.q = s.conv + (inner + G * N) * es;
+    d.ld_q = d.ld_k = d.ld_v = C;
+    d.a_pre = s.proj + l.ra_off * es;
+    d.ld_a = P;
+    d.a_log = l.r_a_log;
+    d.dt_bias = l.r_dt_bias;
+    d.skip = l.r_skip;
+    d.q_scale = 1.f;
+    d.state = l.layer_state + hist;
+    d.state_stride = l.layer_state_stride;
+    d.state_slots = b.state_slots;
+    d.query_start = b.query_start;
+    d.context_lens = b.context_lens;
+    d.out = s.of32;
+    d.T = b.num_tokens;
+    d.B = b.num_seqs;
+    d.H = H;
+    d.G = G;
+    d.dim = N;
+    d.vdim = V;
+    d.dtype = dt;
+    if (!hyb_state_scan(d, stream)) return false;
+    return hyb_gate_groupnorm(s.of32, s.proj + l.rg_off * es, P, l.r_head_norm, s.act + l.r_mix_off * es, l.mix_cols, b.num_tokens, inner, l.r_norm_groups,
+                              l.r_mix_off - l.heads * l.vdim, l.mix_cols - l.r_mix_off - inner, m.eps, dt, stream);
 }
 
 // Latent attention of a post-norm layer: norms, rotation and cache write -> queries into the space of the cached rows -> attention
@@ -1012,7 +1100,8 @@ bool postnorm_lru(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, cons
     return hyb_linear_scan(a, stream);
 }
 
-// One layer of a post-norm design: x <- norm1(alpha x + mixer(x)); x <- norm2(alpha x + ff(x)); then the average over depth.  s.h holds
+// One layer of a post-norm design: x <- norm1(alpha x + mixer(x)); x <- norm2(alpha x + ff(x)); then the average over depth (or, with
+// norm_branch, x <- alpha x + branch_scale norm1(mixer(x)) and so on).  s.h holds
 // x in the activation format on entry and the next layer's on return; the stream itself is s.x.
 bool postnorm_layer(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, const atoma_hybrid_layer &l, int64_t index, const Scratch &s,
                     float *trace, cudaStream_t stream) {
@@ -1022,13 +1111,17 @@ bool postnorm_layer(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, co
     int64_t mixed = l.heads * l.vdim;
     if (l.mixer == ATOMA_MIXER_SOFTMAX_ATTENTION) {
         if (!postnorm_softmax(m, b, l, s, stream)) return false;
+        if (l.diff_gain != 0.f) mixed /= 2;
+    } else if (l.mixer == ATOMA_MIXER_ATTENTION_SSM) {
+        if (!postnorm_softmax(m, b, l, s, stream) || !postnorm_ssm(m, b, l, s, stream)) return false;
+        mixed = l.mix_cols;
     } else if (l.mixer == ATOMA_MIXER_LATENT_ATTENTION) {
         if (!postnorm_latent(m, b, l, s, stream)) return false;
     } else if (l.mixer == ATOMA_MIXER_LRU) {
         if (!postnorm_lru(m, b, l, s, stream)) return false;
         mixed = l.lru_width;
     } else {
-        set_status(kErrUnsupported, "atoma_hybrid_step: post-norm layers take softmax attention, latent attention or the linear recurrent unit, got %d",
+        set_status(kErrUnsupported, "atoma_hybrid_step: post-norm layers take softmax attention (alone or beside a state-space recurrence), latent attention or the linear recurrent unit, got %d",
                    l.mixer);
         return false;
     }
@@ -1044,7 +1137,13 @@ bool postnorm_layer(const atoma_hybrid_model &m, const atoma_hybrid_batch &b, co
     r.eps = m.eps;
     r.weight_offset = m.norm_offset;
     r.dtype = dt;
+    r.norm_branch = m.norm_branch;
+    r.branch_scale = m.branch_scale;
+    r.y_scale = 1.f;
     atoma_postnorm_args f = r;          // the layer's last update
+    r.y_bias = l.b_o;
+    r.y_scale = l.mix_scale;
+    if (!l.has_mlp) f.y_bias = r.y_bias, f.y_scale = r.y_scale;
     f.w_norm = l.has_mlp ? l.norm2 : l.norm1;
     f.depth = l.depth_w ? s.depth : nullptr;
     f.depth_w = l.depth_w;
@@ -1158,12 +1257,18 @@ extern "C" void atoma_hybrid_step(const atoma_hybrid_model *model, const atoma_h
     const float off = m.norm_offset;
     const int64_t groups = m.norm_groups > 0 ? m.norm_groups : 1;
     if (m.block_style == ATOMA_BLOCK_POSTNORM) {
-        // the normed embedding rows are the first row of the average over depth
-        if (!m.embed_norm) {
-            set_status(kErrInvalidArg, "atoma_hybrid_step: a post-norm design needs the norm of the embedding");
+        // the (normed) embedding rows are the first row of the average over depth
+        if (!m.embed_norm && m.layers[0].depth_w) {
+            set_status(kErrInvalidArg, "atoma_hybrid_step: an average over depth needs the norm of the embedding");
             return;
         }
-        if (!hyb_embed_scaled_lanes(b.tokens, m.embed, 1.f, s.x, T, 1, W, m.vocab, dt, stream)) return;
+        if (m.pair_table && !b.prev_tokens) {
+            set_status(kErrInvalidArg, "atoma_hybrid_step: a pair table needs the tokens before the portions");
+            return;
+        }
+        if (!hyb_embed_pairs(b.tokens, b.token_seq, b.query_start, b.prev_tokens, m.embed, m.pair_table, m.pair_buckets, m.pair_mul_prev, m.pair_mul_cur,
+                             s.x, m.embed_norm ? nullptr : s.h, T, W, m.vocab, dt, stream))
+            return;
         atoma_postnorm_args r{};
         r.x = s.x;
         r.w_norm = m.embed_norm;
@@ -1176,7 +1281,7 @@ extern "C" void atoma_hybrid_step(const atoma_hybrid_model *model, const atoma_h
         r.eps = m.eps;
         r.weight_offset = off;
         r.dtype = dt;
-        if (!hyb_postnorm_residual(r, stream)) return;
+        if (m.embed_norm && !hyb_postnorm_residual(r, stream)) return;
         for (int64_t i = 0; i < m.num_layers; ++i) {
             if (!postnorm_layer(m, b, m.layers[i], i, s, b.residual_trace ? b.residual_trace + i * T * W : nullptr, stream)) return;
         }

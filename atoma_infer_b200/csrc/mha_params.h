@@ -47,6 +47,8 @@ struct MhaParams {
     int d_k;
     const void *gate;
     int64_t gate_rs;
+    // tcgen05 prefill kernel only: neighbouring key heads that share one value head (0: 1); v then has h_k / v_share heads per row
+    int v_share;
 };
 
 }  // namespace atoma

@@ -4,7 +4,7 @@
 // causal tap filter over time, and both results join the stream in one update (fused here with whatever precedes the next
 // layer and with its input norm).  The mixers that need more than attention kernels:
 //   - tap filters whose inputs before a portion come from a per-sequence history (the portion's last inputs replace it),
-//   - matrix-state recurrences (gated linear attention, gated delta rule): every head keeps S [dim, vdim] in float32; the
+//   - matrix-state recurrences (gated linear attention, gated delta rule, state-space recurrence): every head keeps S [dim, vdim] in float32; the
 //     columns of S are independent in both recurrences, so a CTA owns 32 columns of one head of one sequence, the rows
 //     of a column are spread over `parts` threads (registers), and the tokens are visited strictly in order,
 //   - rotary positions on queries, keys and values with the cache write, the turn-back of a head's sum, and the
@@ -294,7 +294,7 @@ __global__ void __launch_bounds__(64 * kScanWarps, 2) state_scan_kernel(const at
     if (n <= 0) return;
     const int per_tok = (KIND == 0 ? 3 : 2) * DS + COLS + 4;     // q, k, (decay per channel), v of the CTA's columns, beta and decay
     for (int i = threadIdx.x; i < 2 * chunk * per_tok; i += blockDim.x) sm[i] = 0.f;   // what lies beyond dim stays zero
-    const int kvh = KIND == 1 ? h / (H / static_cast<int>(a.G)) : h;
+    const int kvh = KIND != 0 ? h / (H / static_cast<int>(a.G)) : h;
     const T *qp = static_cast<const T *>(a.q), *kp = static_cast<const T *>(a.k), *vp = static_cast<const T *>(a.v);
     const int jb = blockIdx.x * COLS;
     const bool loader = warp >= kScanWarps;
@@ -308,6 +308,7 @@ __global__ void __launch_bounds__(64 * kScanWarps, 2) state_scan_kernel(const at
     const int vcol = (lane < COLS && jb + lane < V) ? jb + lane : -1;
     float zb[EPL];                                               // what does not change from token to token
     float neg_rate = 0.f, dtb = 0.f;
+    const float skip = KIND == 2 && a.skip ? a.skip[h] : 0.f;
     if (KIND == 0) {
 #pragma unroll
         for (int e = 0; e < EPL; ++e) zb[e] = lane + 32 * e < D ? a.z_bias[h * D + lane + 32 * e] : 0.f;
@@ -333,10 +334,8 @@ __global__ void __launch_bounds__(64 * kScanWarps, 2) state_scan_kernel(const at
                     if (KIND == 0) zr[u][e] = static_cast<const T *>(a.z)[t * a.ld_z + h * D + i];
                 }
                 vr[u] = vp[t * a.ld_v + h * V + max(vcol, 0)];
-                if (KIND == 1) {
-                    br[u] = static_cast<const T *>(a.b_pre)[t * a.ld_b + h];
-                    ar[u] = static_cast<const T *>(a.a_pre)[t * a.ld_a + h];
-                }
+                if (KIND == 1) br[u] = static_cast<const T *>(a.b_pre)[t * a.ld_b + h];
+                if (KIND != 0) ar[u] = static_cast<const T *>(a.a_pre)[t * a.ld_a + h];
             }
 #pragma unroll
             for (int u = 0; u < TU; ++u) {
@@ -370,6 +369,11 @@ __global__ void __launch_bounds__(64 * kScanWarps, 2) state_scan_kernel(const at
                     if (KIND == 1) {
                         row[per_tok - 4] = sigmoidf_(to_f(br[u]));
                         row[per_tok - 3] = expf(neg_rate * softplusf_(to_f(ar[u]) + dtb));
+                    }
+                    if (KIND == 2) {
+                        const float step = softplusf_(to_f(ar[u]) + dtb);
+                        row[per_tok - 4] = step;
+                        row[per_tok - 3] = expf(neg_rate * step);
                     }
                     row[per_tok - 2] = dot * fq * fk;            // q . k of the token as the recurrence sees them
                 }
@@ -453,6 +457,31 @@ __global__ void __launch_bounds__(64 * kScanWarps, 2) state_scan_kernel(const at
 #pragma unroll
                         for (int g8 = 0; g8 < G8; g8 += 2 * w) gs[g8] += gs[g8 + w];
                     o = fmaf(kq, vj, parts_sum<PW>(gs[0]));
+                } else if (KIND == 2) {
+                    const float g = row[per_tok - 3], u = row[per_tok - 4] * vj;   // decay, written row
+                    float gs[G8];
+#pragma unroll
+                    for (int g8 = 0; g8 < G8; ++g8) {
+                        float c[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                        for (int r4 = 2 * g8; r4 < 2 * g8 + 2; ++r4) {
+                            const float4 k4 = kr[r4], q4 = qr[r4];
+                            c[0] = fmaf(S[4 * r4], q4.x, c[0]);
+                            S[4 * r4] = fmaf(g, S[4 * r4], k4.x * u);
+                            c[1] = fmaf(S[4 * r4 + 1], q4.y, c[1]);
+                            S[4 * r4 + 1] = fmaf(g, S[4 * r4 + 1], k4.y * u);
+                            c[2] = fmaf(S[4 * r4 + 2], q4.z, c[2]);
+                            S[4 * r4 + 2] = fmaf(g, S[4 * r4 + 2], k4.z * u);
+                            c[3] = fmaf(S[4 * r4 + 3], q4.w, c[3]);
+                            S[4 * r4 + 3] = fmaf(g, S[4 * r4 + 3], k4.w * u);
+                        }
+                        gs[g8] = (c[0] + c[1]) + (c[2] + c[3]);
+                    }
+#pragma unroll
+                    for (int w = 1; w < G8; w <<= 1)
+#pragma unroll
+                        for (int g8 = 0; g8 < G8; g8 += 2 * w) gs[g8] += gs[g8 + w];
+                    o = fmaf(g, parts_sum<PW>(gs[0]), fmaf(kq, u, skip * vj));
                 } else {
                     const float beta = row[per_tok - 4], g = row[per_tok - 3];
                     float gk[G8], gq[G8];
@@ -553,15 +582,14 @@ __device__ __forceinline__ void turn(float pos, float freq, float freq_lo, float
     cs = amplitude * fmaf(-rest, s, c * near_one);
 }
 
-// buf [n] float32 (one warp's): the first 2 pairs entries turned by sign * pos * freq, written to dst as T.
+// buf [n] float32 (one warp's): the first 2 pairs entries turned by pos * freq, written to dst as T.
 template <typename T>
-__device__ __forceinline__ void rotate_store(const float *buf, int n, const float *__restrict__ freq, int pairs, int interleaved, float pos,
-                                             float sign, T *__restrict__ dst, int lane) {
+__device__ __forceinline__ void rotate_store(const float *buf, int n, const float *__restrict__ freq, const float *__restrict__ freq_lo, float amplitude,
+                                             int pairs, int interleaved, float pos, T *__restrict__ dst, int lane) {
     for (int i = lane; i < pairs; i += 32) {
         const int ia = interleaved ? 2 * i : i, ib = interleaved ? 2 * i + 1 : i + pairs;
         float sn, cs;
-        sincosf(pos * freq[i], &sn, &cs);
-        sn *= sign;
+        turn(pos, freq[i], freq_lo ? freq_lo[i] : 0.f, amplitude, sn, cs);
         const float u = buf[ia], v = buf[ib];
         dst[ia] = from_f<T>(u * cs - v * sn);
         dst[ib] = from_f<T>(v * cs + u * sn);
@@ -577,12 +605,15 @@ __global__ void __launch_bounds__(256) qkv_headnorm_rope_cache_kernel(const atom
     const int64_t t = blockIdx.x;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
     const int H = static_cast<int>(a.H), G = static_cast<int>(a.G), D = static_cast<int>(a.dim), V = static_cast<int>(a.vdim);
+    const int Gv = a.v_heads > 0 ? static_cast<int>(a.v_heads) : G;
+    const int units = a.slot_mapping ? H + G + Gv : H;
+    const float amplitude = a.qk_amplitude != 0.f ? a.qk_amplitude : 1.f;
     const int wide = max(D, V);
     float *buf = sm + warp * wide;
     const T *row = static_cast<const T *>(a.proj) + t * a.ld;
     const float pos = static_cast<float>(a.positions[t]);
     const int64_t slot = a.slot_mapping ? a.slot_mapping[t] : -1;
-    for (int u = warp; u < H + 2 * G; u += nwarp) {
+    for (int u = warp; u < units; u += nwarp) {
         const bool is_q = u < H, is_k = !is_q && u < H + G;
         const int hd = is_q ? u : (is_k ? u - H : u - H - G);
         if (!is_q && slot < 0) continue;
@@ -606,11 +637,11 @@ __global__ void __launch_bounds__(256) qkv_headnorm_rope_cache_kernel(const atom
         }
         __syncwarp();
         T *dst = is_q ? static_cast<T *>(a.q_out) + (t * H + hd) * D
-                      : (is_k ? static_cast<T *>(a.k_cache) + (slot * G + hd) * D : static_cast<T *>(a.v_cache) + (slot * G + hd) * V);
+                      : (is_k ? static_cast<T *>(a.k_cache) + (slot * G + hd) * D : static_cast<T *>(a.v_cache) + (slot * Gv + hd) * V);
         const bool vpart = !is_q && !is_k;
         const float *freq = vpart ? a.v_freq : a.qk_freq;
         const int pairs = freq ? static_cast<int>(vpart ? a.v_pairs : a.rot_pairs) : 0;
-        rotate_store<T>(buf, n, freq, pairs, a.interleaved, pos, 1.f, dst, lane);
+        rotate_store<T>(buf, n, freq, vpart ? nullptr : a.qk_freq_lo, vpart ? 1.f : amplitude, pairs, a.interleaved, pos, dst, lane);
         __syncwarp();
     }
 }
@@ -771,10 +802,11 @@ bool hyb_tap_filter(const atoma_tap_filter_args &a, cudaStream_t stream) {
 bool hyb_state_scan(const atoma_state_scan_args &a, cudaStream_t stream) {
     if (a.T <= 0 || a.B <= 0) return true;
     if (!hybrid::known_dtype(a.dtype, "atoma_state_scan")) return false;
-    const bool gla = a.kind == 0, delta = a.kind == 1;
-    if ((!gla && !delta) || !a.q || !a.k || !a.v || !a.state || !a.state_slots || !a.query_start || !a.context_lens || !a.out || a.H <= 0 ||
+    const bool gla = a.kind == 0, delta = a.kind == 1, ssm = a.kind == 2;
+    if ((!gla && !delta && !ssm) || !a.q || !a.k || !a.v || !a.state || !a.state_slots || !a.query_start || !a.context_lens || !a.out || a.H <= 0 ||
         a.dim <= 0 || a.vdim <= 0 || a.state_stride < a.H * a.dim * a.vdim || (gla && (!a.z || !a.z_bias || !(a.tau > 0.f))) ||
-        (delta && (!a.b_pre || !a.a_pre || !a.a_log || !a.dt_bias || a.G <= 0 || a.H % a.G))) {
+        (delta && !a.b_pre) ||
+        (!gla && (!a.a_pre || !a.a_log || !a.dt_bias || a.G <= 0 || a.H % a.G))) {
         set_status(kErrInvalidArg, "atoma_state_scan: null argument, unknown kind %d, or a state row shorter than heads * dim * vdim", a.kind);
         return false;
     }
@@ -821,6 +853,7 @@ bool hyb_state_scan(const atoma_state_scan_args &a, cudaStream_t stream) {
 #define SCAN_T(TT)                                      \
     do {                                                \
         if (gla) SCAN_K(TT, 0);                         \
+        else if (ssm) SCAN_K(TT, 2);                    \
         else SCAN_K(TT, 1);                             \
     } while (0)
     if (a.dtype == ATOMA_DTYPE_BF16) SCAN_T(__nv_bfloat16);
@@ -850,8 +883,8 @@ bool hyb_qkv_headnorm_rope_cache(const atoma_qkv_rope_args &a, cudaStream_t stre
     if (a.T <= 0) return true;
     if (!hybrid::known_dtype(a.dtype, "atoma_qkv_headnorm_rope_cache")) return false;
     if (!a.proj || !a.q_out || !a.positions || a.H <= 0 || a.G <= 0 || a.H % a.G || a.dim <= 0 || a.vdim <= 0 ||
-        (a.slot_mapping && (!a.k_cache || !a.v_cache)) || a.q_off < 0 || a.k_off < 0 || a.v_off < 0 || a.q_off + a.H * a.dim > a.ld ||
-        a.k_off + a.G * a.dim > a.ld || a.v_off + a.G * a.vdim > a.ld || a.rot_pairs < 0 || 2 * a.rot_pairs > a.dim || a.v_pairs < 0 ||
+        (a.slot_mapping && (!a.k_cache || !a.v_cache)) || a.q_off < 0 || (a.slot_mapping && (a.k_off < 0 || a.v_off < 0)) || a.q_off + a.H * a.dim > a.ld ||
+        (a.slot_mapping && (a.k_off + a.G * a.dim > a.ld || a.v_off + (a.v_heads > 0 ? a.v_heads : a.G) * a.vdim > a.ld)) || a.v_heads < 0 || a.rot_pairs < 0 || 2 * a.rot_pairs > a.dim || a.v_pairs < 0 ||
         2 * a.v_pairs > a.vdim || (a.rot_pairs > 0 && !a.qk_freq) || (a.q_head_scale && !a.q_weight && !a.unit_norm)) {
         set_status(kErrInvalidArg, "atoma_qkv_headnorm_rope_cache: null argument, columns outside the row, or more rotated entries than a head has");
         return false;

@@ -4,6 +4,7 @@
 // may become a weighted average over DEPTH: of the embedding output and of every layer's result so far, which are kept as float32
 // rows [layer][token][width] for the step.  One CTA per token does the sum (with the token's routed experts' rows), the norm, the
 // write of the layer's row, the average, and the copy in the activation format that the next sublayer's projections read.
+// A second form norms the sublayer's result instead of the sum and adds it to the stream (norm_branch).
 // Everything is float32; rows are reduced in an order that depends on the row alone.
 #include "common.cuh"
 #include "hybrid_common.cuh"
@@ -73,13 +74,28 @@ __global__ void __launch_bounds__(kRowThreads) postnorm_residual_kernel(const at
     float ss = 0.f;
     for (int c = C * threadIdx.x; c < W; c += C * blockDim.x) {
         float v[C], s[C];
-        Q::load(x + c, v);
+        if (a.norm_branch) {
 #pragma unroll
-        for (int i = 0; i < C; ++i) v[i] *= a.alpha;
-        if (y) {
-            Q::load(y + c, s);
+            for (int i = 0; i < C; ++i) v[i] = 0.f;
+            if (y) {
+                Q::load(y + c, s);
 #pragma unroll
-            for (int i = 0; i < C; ++i) v[i] += s[i];
+                for (int i = 0; i < C; ++i) v[i] = a.y_scale * s[i];
+            }
+            if (a.y_bias) {
+                Q::load(a.y_bias + c, s);
+#pragma unroll
+                for (int i = 0; i < C; ++i) v[i] += s[i];
+            }
+        } else {
+            Q::load(x + c, v);
+#pragma unroll
+            for (int i = 0; i < C; ++i) v[i] *= a.alpha;
+            if (y) {
+                Q::load(y + c, s);
+#pragma unroll
+                for (int i = 0; i < C; ++i) v[i] += s[i];
+            }
         }
         for (int k = 0; k < top; ++k) {
             if (erow[k] < 0) continue;
@@ -103,6 +119,12 @@ __global__ void __launch_bounds__(kRowThreads) postnorm_residual_kernel(const at
         Q::load(a.w_norm + c, w);
 #pragma unroll
         for (int i = 0; i < C; ++i) n[i] = row[c + i] * inv * (a.weight_offset + w[i]);
+        if (a.norm_branch) {
+            float s[C];
+            Q::load(x + c, s);
+#pragma unroll
+            for (int i = 0; i < C; ++i) n[i] = fmaf(a.branch_scale, n[i], a.alpha * s[i]);
+        }
         if (nd > 0) {
             float *d = a.depth + t * W + c;
             Q::store(d + (nd - 1) * plane, n);
@@ -150,7 +172,7 @@ bool hyb_postnorm_residual(const atoma_postnorm_args &a, cudaStream_t stream) {
         return false;
     }
     auto al = [](const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    const bool vec = a.width % 4 == 0 && al(a.x) && al(a.y) && al(a.expert_out) && al(a.w_norm) && al(a.depth) && al(a.h) && al(a.trace);
+    const bool vec = a.width % 4 == 0 && al(a.x) && al(a.y) && al(a.expert_out) && al(a.w_norm) && al(a.y_bias) && al(a.depth) && al(a.h) && al(a.trace);
     cudaError_t e;
 #define CASE(TT, V)                                                                                                                       \
     {                                                                                                                                     \

@@ -227,7 +227,8 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
             const int d_k = p.d_k > 0 ? p.d_k : D;
             const T *qg = static_cast<const T *>(p.q) + si.q_off + static_cast<int64_t>(head) * p.q_hs;
             const T *kg = static_cast<const T *>(p.k) + si.k_off + static_cast<int64_t>(kvh) * p.k_hs;
-            const T *vg = static_cast<const T *>(p.v) + si.v_off + static_cast<int64_t>(kvh) * p.v_hs;
+            const int vh = p.v_share > 1 ? kvh / p.v_share : kvh;
+            const T *vg = static_cast<const T *>(p.v) + si.v_off + static_cast<int64_t>(vh) * p.v_hs;
 #pragma unroll
             for (int t = 0; t < kQTiles; ++t)
                 if (nt[t] > 0)
@@ -242,7 +243,7 @@ prefill_attn_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_cons
                 ++k_issued;
                 if (!pf_wait_all(&v_empty[vs], ((jj / kVStages) & 1) ^ 1, late)) break;
                 load_tile(VPieces(), D, sv + vs * C::kVBytes, &map_v, &v_full[vs], vg, p.v_rs, j * kPfN, len_k,
-                          si.k_row0 + j * kPfN, kvh, si.k_batch, kL2EvictLast);
+                          si.k_row0 + j * kPfN, vh, si.k_batch, kL2EvictLast);
                 ++v_issued;
             }
             // whatever happens to the other roles, the copies have landed before this warp leaves
@@ -613,9 +614,11 @@ int try_launch_prefill_tc(const MhaParams &p, bool is_bf16, cudaStream_t stream)
     const int d_k = p.d_k > 0 ? p.d_k : p.d;
     if (!make_attn_map(&mq, p.q, d_k, p.h, q_rows, q_b, p.q_hs, p.q_rs, q_bs, is_bf16)) return -1;
     if (!make_attn_map(&mk, p.k, d_k, p.h_k, k_rows, k_b, p.k_hs, p.k_rs, k_bs, is_bf16)) return -1;
-    if (!make_attn_map(&mv, p.v, p.d, p.h_k, k_rows, k_b, p.v_hs, p.v_rs, v_bs, is_bf16)) return -1;
+    if (!make_attn_map(&mv, p.v, p.d, p.v_share > 1 ? p.h_k / p.v_share : p.h_k, k_rows, k_b, p.v_hs, p.v_rs, v_bs, is_bf16)) return -1;
     bool ok;
-    if ((d_k + 63) / 64 > p.d / 64)   // longer query / key heads than value heads
+    if (p.d == 128 && d_k <= 64 && is_bf16 && !p.dist_bias)   // shorter query / key heads: one 64-column piece
+        ok = launch_prefill_b<__nv_bfloat16, 128, 1, false>(mq, mk, mv, p, stream);
+    else if ((d_k + 63) / 64 > p.d / 64)   // longer query / key heads than value heads
         ok = p.d == 128 ? launch_prefill_b<__nv_bfloat16, 128, 3, false>(mq, mk, mv, p, stream)
                         : launch_prefill_b<__nv_bfloat16, 64, 2, false>(mq, mk, mv, p, stream);
     else if (is_bf16) ok = p.d == 128 ? launch_prefill<__nv_bfloat16, 128>(mq, mk, mv, p, stream)

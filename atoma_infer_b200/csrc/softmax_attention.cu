@@ -54,6 +54,7 @@ __global__ void __launch_bounds__(kGenThreads) softmax_attn_general_kernel(const
     pdl_wait();
     const int H = static_cast<int>(a.H), G = static_cast<int>(a.G), D = static_cast<int>(a.dim), Dv = static_cast<int>(a.vdim);
     const int t = blockIdx.x, h = blockIdx.y, g = h / (H / G);
+    const int share = a.v_share > 1 ? static_cast<int>(a.v_share) : 1, gv = g / share, Gv = G / share;
     const int b = a.token_seq[t];
     if (a.skip_min_q > 0 && a.query_start && a.query_start[b + 1] - a.query_start[b] >= a.skip_min_q) return;
     const int p = static_cast<int>(a.positions[t]);
@@ -101,14 +102,14 @@ __global__ void __launch_bounds__(kGenThreads) softmax_attn_general_kernel(const
             const int d = threadIdx.x + r * kGenThreads;
             if (d < Dv) {
                 float o = acc[r] * corr;
-                for (int jj = 0; jj < nj; ++jj) o = fmaf(w_s[jj], to_f(vc[(slot_s[jj] * G + g) * Dv + d]), o);
+                for (int jj = 0; jj < nj; ++jj) o = fmaf(w_s[jj], to_f(vc[(slot_s[jj] * Gv + gv) * Dv + d]), o);
                 acc[r] = o;
             }
         }
         __syncthreads();
     }
     const float inv = 1.0f / l_run;
-    T *o = static_cast<T *>(a.out) + (static_cast<int64_t>(t) * H + h) * Dv;
+    T *o = static_cast<T *>(a.out) + static_cast<int64_t>(t) * a.ld_out + h * Dv;
     const T *gt = a.gate ? static_cast<const T *>(a.gate) + static_cast<int64_t>(t) * a.ld_gate + h * Dv : nullptr;
 #pragma unroll
     for (int r = 0; r < kGenOut; ++r) {
@@ -125,13 +126,16 @@ __global__ void __launch_bounds__(kGenThreads) softmax_attn_general_kernel(const
 
 #define HYB_DISPATCH(dtype, CALL) ((dtype) == ATOMA_DTYPE_BF16 ? CALL(__nv_bfloat16) : CALL(float))
 
-bool hyb_softmax_attention(const atoma_softmax_attn_args &a, cudaStream_t stream) {
+bool hyb_softmax_attention(const atoma_softmax_attn_args &args, cudaStream_t stream) {
+    atoma_softmax_attn_args a = args;
+    if (a.ld_out == 0) a.ld_out = a.H * a.vdim;
+    if (a.v_share == 0) a.v_share = 1;
     if (a.T <= 0) return true;
     if (!hybrid::known_dtype(a.dtype, "atoma_softmax_attention_paged")) return false;
     if (!a.q || !a.k_cache || !a.v_cache || !a.out || !a.positions || !a.token_seq || !a.block_tables || a.H <= 0 || a.G <= 0 || a.H % a.G ||
         a.dim <= 0 || a.vdim <= 0 || a.block_size <= 0 || a.max_blocks <= 0 || (a.dist_bias && a.dist_rows <= 0) ||
-        (a.gate && a.ld_gate < a.H * a.vdim)) {
-        set_status(kErrInvalidArg, "atoma_softmax_attention_paged: null argument, inconsistent head counts, an empty distance table or a gate row shorter than the heads");
+        (a.gate && a.ld_gate < a.H * a.vdim) || a.ld_out < a.H * a.vdim || a.v_share < 0 || a.G % a.v_share) {
+        set_status(kErrInvalidArg, "atoma_softmax_attention_paged: null argument, inconsistent head counts, an empty distance table, a gate or output row shorter than the heads, or key heads that do not share value heads evenly");
         return false;
     }
     if (a.skip_min_q == 0 && hyb_softmax_long_ok(a)) {

@@ -1,5 +1,6 @@
 // Softmax attention for LONG prompt portions on the tensor-memory prefill kernel (include/atoma_hybrid.h,
-// atoma_softmax_attention_paged with long_seqs > 0): bfloat16 heads of 64 or 128, dim = vdim.
+// atoma_softmax_attention_paged with long_seqs > 0): bfloat16 heads of 64 or 128, dim = vdim; without a table, kept tokens and a gate
+// also value heads of 64 or 128 with key heads of another size, and key heads that share value heads.
 //
 // For every sequence with at least long_min_q query tokens in the step:
 //   1. softmax_long_plan_kernel fixes, on the device, the first key the portion's first query sees through the window and the
@@ -50,11 +51,12 @@ __global__ void softmax_long_plan_kernel(const int32_t *__restrict__ query_start
     cu_k[B] = acc;
 }
 
-// One warp per gathered key: its row of the key cache and of the value cache (all key/value heads, `row` elements each).
+// One warp per gathered key: its row of the key cache and of the value cache (all heads: k_row and v_row elements).
 __global__ void __launch_bounds__(256) paged_kv_gather_kernel(const __nv_bfloat16 *__restrict__ k_cache, const __nv_bfloat16 *__restrict__ v_cache,
                                                               const int32_t *__restrict__ block_tables, int64_t max_blocks,
                                                               const int32_t *__restrict__ cu_k, const int32_t *__restrict__ key_lo,
-                                                              __nv_bfloat16 *__restrict__ k_out, __nv_bfloat16 *__restrict__ v_out, int row, int bs) {
+                                                              __nv_bfloat16 *__restrict__ k_out, __nv_bfloat16 *__restrict__ v_out, int k_row, int v_row,
+                                                              int bs) {
     pdl_launch_dependents();
     pdl_wait();
     const int b = blockIdx.y;
@@ -63,12 +65,13 @@ __global__ void __launch_bounds__(256) paged_kv_gather_kernel(const __nv_bfloat1
     if (i >= n) return;
     const int j = key_lo[b] + i;
     const int32_t *bt = block_tables + static_cast<int64_t>(b) * max_blocks;
-    const int64_t slot = static_cast<int64_t>(bt[j / bs]) * bs + j % bs, dst = static_cast<int64_t>(cu_k[b] + i) * row;
-    const uint4 *ks = reinterpret_cast<const uint4 *>(k_cache + slot * row), *vs = reinterpret_cast<const uint4 *>(v_cache + slot * row);
-    uint4 *kd = reinterpret_cast<uint4 *>(k_out + dst), *vd = reinterpret_cast<uint4 *>(v_out + dst);
-    for (int c = threadIdx.x & 31; c < row / 8; c += 32) {
-        kd[c] = ks[c];
-        vd[c] = vs[c];
+    const int64_t slot = static_cast<int64_t>(bt[j / bs]) * bs + j % bs, dst = static_cast<int64_t>(cu_k[b] + i);
+    const uint4 *ks = reinterpret_cast<const uint4 *>(k_cache + slot * k_row), *vs = reinterpret_cast<const uint4 *>(v_cache + slot * v_row);
+    uint4 *kd = reinterpret_cast<uint4 *>(k_out + dst * k_row), *vd = reinterpret_cast<uint4 *>(v_out + dst * v_row);
+    const int lane = threadIdx.x & 31, nk = k_row / 8, nv = v_row / 8;
+    for (int c = lane; c < max(nk, nv); c += 32) {
+        if (c < nk) kd[c] = ks[c];
+        if (c < nv) vd[c] = vs[c];
     }
 }
 
@@ -102,7 +105,7 @@ __global__ void __launch_bounds__(128) softmax_kept_merge_gate_kernel(const atom
     const int lo = a.window > 0 ? max(0, p - static_cast<int>(a.window) + 1) : 0;
     const int kept = a.keep_first <= 0 ? 0 : (a.keep_first < lo ? static_cast<int>(a.keep_first) : lo);
     const int c0 = lane * PER;   // this lane's channels
-    __nv_bfloat16 *out = static_cast<__nv_bfloat16 *>(a.out) + (t * H + h) * D + c0;
+    __nv_bfloat16 *out = static_cast<__nv_bfloat16 *>(a.out) + t * a.ld_out + h * D + c0;
     float o[PER];
     load_row<PER>(out, o);
     if (kept > 0) {
@@ -159,27 +162,30 @@ __global__ void __launch_bounds__(128) softmax_kept_merge_gate_kernel(const atom
 
 }  // namespace
 
-// Shapes the long-portion path takes: bfloat16, equal key and value head sizes of 64 or 128, sm_100.
+// Shapes the long-portion path takes: bfloat16, value heads of 64 or 128, key heads of the same size (or, in the plain form, of any
+// multiple of 8 the prefill kernel takes), sm_100.
 bool hyb_softmax_long_ok(const atoma_softmax_attn_args &a) {
     auto al = [](const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    return a.dtype == ATOMA_DTYPE_BF16 && a.dim == a.vdim && (a.dim == 64 || a.dim == 128) && a.long_seqs > 0 && a.long_min_q >= 32 &&
-           a.query_start && al(a.q) && al(a.out) && al(a.k_cache) && al(a.v_cache) && (!a.gate || (al(a.gate) && a.ld_gate % 8 == 0)) && a.scale > 0.f && a.T < (1ll << 26) &&
-           current_device_info().cc_major == 10 && !(g_hybrid_debug & 2);
+    const bool plain = !a.dist_bias && !a.gate && (a.keep_first <= 0 || a.window <= 0);
+    const bool sizes = a.dim == a.vdim ? (plain || a.v_share == 1) : (plain && a.dim % 8 == 0 && a.dim <= a.vdim + 64);
+    return a.dtype == ATOMA_DTYPE_BF16 && (a.vdim == 64 || a.vdim == 128) && sizes && a.long_seqs > 0 && a.long_min_q >= 32 &&
+           a.query_start && al(a.q) && al(a.out) && a.ld_out % 8 == 0 && al(a.k_cache) && al(a.v_cache) && (!a.gate || (al(a.gate) && a.ld_gate % 8 == 0)) &&
+           a.scale > 0.f && a.T < (1ll << 26) && current_device_info().cc_major == 10 && !(g_hybrid_debug & 2);
 }
 
 bool hyb_softmax_attention_long(const atoma_softmax_attn_args &a, cudaStream_t stream) {
-    const int64_t row = a.G * a.dim, HD = a.H * a.dim;
+    const int64_t k_row = a.G * a.dim, v_row = a.G / a.v_share * a.vdim;
     const int64_t kept_ctx = a.window > 0 ? std::min<int64_t>(a.long_ctx_sum, static_cast<int64_t>(a.long_seqs) * (a.window - 1)) : a.long_ctx_sum;
     const int64_t max_keys = a.long_tokens + kept_ctx;
     if (max_keys <= 0) return true;
     auto up = [](int64_t x) { return (x + 255) / 256 * 256; };
     const int64_t rows = max_keys + 128;   // the attention kernel's TMA boxes may start up to a tile before the end
-    const int64_t b_int = up((2 * a.B + 2) * 4), b_kv = up(rows * row * 2), b_lse = up(a.H * a.T * 4);
-    char *ws = static_cast<char *>(get_workspace(stream, static_cast<size_t>(b_int + 2 * b_kv + b_lse), kWorkspaceLatentExpand));
+    const int64_t b_int = up((2 * a.B + 2) * 4), b_k = up(rows * k_row * 2), b_v = up(rows * v_row * 2), b_lse = up(a.H * a.T * 4);
+    char *ws = static_cast<char *>(get_workspace(stream, static_cast<size_t>(b_int + b_k + b_v + b_lse), kWorkspaceLatentExpand));
     if (!ws) return false;
     int32_t *cu_k = reinterpret_cast<int32_t *>(ws), *key_lo = cu_k + a.B + 1;
-    __nv_bfloat16 *K = reinterpret_cast<__nv_bfloat16 *>(ws + b_int), *V = reinterpret_cast<__nv_bfloat16 *>(ws + b_int + b_kv);
-    float *lse = reinterpret_cast<float *>(ws + b_int + 2 * b_kv);
+    __nv_bfloat16 *K = reinterpret_cast<__nv_bfloat16 *>(ws + b_int), *V = reinterpret_cast<__nv_bfloat16 *>(ws + b_int + b_k);
+    float *lse = reinterpret_cast<float *>(ws + b_int + b_k + b_v);
     if (!hybrid::launched(launch_ex(softmax_long_plan_kernel, dim3(1), dim3(32), 0, stream, a.query_start, a.positions, static_cast<int>(a.B),
                                     static_cast<int>(std::min<int64_t>(a.window, 0x3fffffff)), static_cast<int>(a.long_min_q), cu_k, key_lo),
                           "softmax_long_plan_kernel"))
@@ -188,16 +194,18 @@ bool hyb_softmax_attention_long(const atoma_softmax_attn_args &a, cudaStream_t s
     const dim3 gg(static_cast<unsigned>((span + 7) / 8), static_cast<unsigned>(a.B));
     if (!hybrid::launched(launch_ex(paged_kv_gather_kernel, gg, dim3(256), 0, stream, static_cast<const __nv_bfloat16 *>(a.k_cache),
                                     static_cast<const __nv_bfloat16 *>(a.v_cache), a.block_tables, a.max_blocks, static_cast<const int32_t *>(cu_k),
-                                    static_cast<const int32_t *>(key_lo), K, V, static_cast<int>(row), static_cast<int>(a.block_size)),
+                                    static_cast<const int32_t *>(key_lo), K, V, static_cast<int>(k_row), static_cast<int>(v_row), static_cast<int>(a.block_size)),
                           "paged_kv_gather_kernel"))
         return false;
     MhaParams p;
     std::memset(&p, 0, sizeof(p));
     p.q = a.q, p.k = K, p.v = V, p.o = a.out, p.lse = lse;
     p.cu_q = a.query_start, p.cu_k = cu_k;
-    p.q_rs = p.o_rs = HD, p.k_rs = p.v_rs = row;
-    p.q_hs = p.k_hs = p.v_hs = p.o_hs = a.dim;
-    p.b = static_cast<int>(a.B), p.h = static_cast<int>(a.H), p.h_k = static_cast<int>(a.G), p.d = static_cast<int>(a.dim);
+    p.q_rs = a.H * a.dim, p.o_rs = a.ld_out, p.k_rs = k_row, p.v_rs = v_row;
+    p.q_hs = p.k_hs = a.dim, p.v_hs = p.o_hs = a.vdim;
+    p.b = static_cast<int>(a.B), p.h = static_cast<int>(a.H), p.h_k = static_cast<int>(a.G), p.d = static_cast<int>(a.vdim);
+    p.d_k = a.dim == a.vdim ? 0 : static_cast<int>(a.dim);
+    p.v_share = static_cast<int>(a.v_share);
     p.seqlen_q = a.max_query_len, p.seqlen_k = static_cast<int>(span);
     p.page = 1;
     p.scale = a.scale, p.scale_log2 = a.scale * 1.4426950408889634f;

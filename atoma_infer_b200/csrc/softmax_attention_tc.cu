@@ -53,10 +53,11 @@ __host__ __device__ inline TcLayout tc_layout(int D, int DV, int bias_n) {
     return l;
 }
 
-// EXACT: dim = vdim = DMAX (the usual case): strides and loop bounds are compile-time constants.
+// DK, DV_MAX: the head sizes rounded up to 64 or 128.  EXACT: dim = DK, vdim = DV_MAX (the usual case): strides and loop bounds are
+// compile-time constants.
 // SIG: the weight of a visible key is sigmoid(score * scale + head_bias[h]) and nothing is normalised (no running maximum, no
 // denominator, no rescaling: the outputs are plain sums) — the same tiles, staging and products serve both kinds of attention.
-template <int DMAX, bool ROWS_ARE_HEADS, bool EXACT, bool SIG>
+template <int DK, int DV_MAX, bool ROWS_ARE_HEADS, bool EXACT, bool SIG>
 __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_softmax_attn_args a, int bias_n, int splits, float *__restrict__ partial,
                                                                  const float *__restrict__ head_bias) {
     extern __shared__ __align__(16) unsigned char smem[];
@@ -64,8 +65,9 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
     pdl_wait();
     constexpr int NT = ROWS_ARE_HEADS ? 2 : kKeys / 8;   // 8-key score tiles per warp and key tile
     const int H = static_cast<int>(a.H), G = static_cast<int>(a.G);
-    const int D = EXACT ? DMAX : static_cast<int>(a.dim), DV = EXACT ? DMAX : static_cast<int>(a.vdim);
+    const int D = EXACT ? DK : static_cast<int>(a.dim), DV = EXACT ? DV_MAX : static_cast<int>(a.vdim);
     const int rep = H / G;
+    const int share = static_cast<int>(a.v_share);
     const int b = blockIdx.y;
     const int t_begin = a.query_start[b], n_q = a.query_start[b + 1] - t_begin;
     if (ROWS_ARE_HEADS ? n_q != 1 : n_q <= 1) return;   // single tokens are served by the rows-are-heads mapping
@@ -102,8 +104,9 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
     __nv_bfloat16 *Vs0 = reinterpret_cast<__nv_bfloat16 *>(smem + L.v_off);
     float *bias_s = reinterpret_cast<float *>(smem + L.bias_off);
     const int k_stage = kKeys * (D + 8), v_stage = kKeys * (DV + 8);
-    const __nv_bfloat16 *kc = static_cast<const __nv_bfloat16 *>(a.k_cache);
-    const __nv_bfloat16 *vc = static_cast<const __nv_bfloat16 *>(a.v_cache);
+    const __nv_bfloat16 *kc = static_cast<const __nv_bfloat16 *>(a.k_cache) + g * D;
+    const __nv_bfloat16 *vc = static_cast<const __nv_bfloat16 *>(a.v_cache) + (g / share) * DV;
+    const int64_t k_row = static_cast<int64_t>(G) * D, v_row = static_cast<int64_t>(G / share) * DV;
     const int last_row = static_cast<int>(a.dist_rows) - 1;
     if constexpr (!ROWS_ARE_HEADS) {
         for (int i = threadIdx.x; i < bias_n; i += blockDim.x) bias_s[i] = a.dist_bias[static_cast<int64_t>(i) * H + h0] * kLog2e;
@@ -123,13 +126,13 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
     auto tile_of = [&](int i) { return i < ka ? i : kt_lo + (i - ka); };
 
     // query fragments (A operand: rows rq / rq + 8, k = 2 t4 .. + 1 and + 8)
-    uint32_t qf[DMAX / 16][4];
+    uint32_t qf[DK / 16][4];
     {
         const __nv_bfloat16 *q = static_cast<const __nv_bfloat16 *>(a.q);
         const int64_t row_stride = ROWS_ARE_HEADS ? D : static_cast<int64_t>(H) * D;
         const __nv_bfloat16 *q0 = q + (static_cast<int64_t>(tok0) * H + h0) * D;
 #pragma unroll
-        for (int kk = 0; kk < DMAX / 16; ++kk) {
+        for (int kk = 0; kk < DK / 16; ++kk) {
             qf[kk][0] = qf[kk][1] = qf[kk][2] = qf[kk][3] = 0u;
             if (kk * 16 < D) {
                 const int col = kk * 16 + 2 * t4;
@@ -144,9 +147,9 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
             }
         }
     }
-    float o[DMAX / 8][4];
+    float o[DV_MAX / 8][4];
 #pragma unroll
-    for (int i = 0; i < DMAX / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+    for (int i = 0; i < DV_MAX / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
     const float scale2 = a.scale * kLog2e;
     float hb[2] = {0.f, 0.f};                                  // SIG: the bias of the head of rows rq and rq + 8, in log2 units
@@ -161,13 +164,13 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
         }
     }
 
-    // cache rows (of the CTA's key/value head) of a tile's keys, looked up once per key one tile ahead of the copies that use
+    // cache rows of a tile's keys, looked up once per key one tile ahead of the copies that use
     // them (-1: past the last key)
     __shared__ int64_t slot_s[2][kKeys];
-    auto slot_of = [&](int i) -> int64_t {     // thread t < 64: the cache row of key t of tile i, (slot * G + g)
+    auto slot_of = [&](int i) -> int64_t {     // thread t < 64: the cache row of key t of tile i
         if (threadIdx.x >= kKeys) return -1;
         const int j = tile_of(i) * kKeys + threadIdx.x;
-        return j <= p_last ? (static_cast<int64_t>(bt[j / bs]) * bs + j % bs) * G + g : -1;
+        return j <= p_last ? static_cast<int64_t>(bt[j / bs]) * bs + j % bs : -1;
     };
     auto fill_slots = [&](int i, int buf) {
         const int64_t v = slot_of(i);
@@ -181,13 +184,13 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
         const int64_t *slots = slot_s[buf];
         for (int jj = k_jj0, e = k_e0; jj < kKeys;) {     // thread -> pieces threadIdx.x, + 128, ... of the tile, (row, piece) kept incrementally
             const int64_t slot = slots[jj];
-            cp_async_16(smem_u32(Kd + jj * (D + 8) + e * 8), kc + (slot < 0 ? 0 : slot) * D + e * 8, slot < 0 ? 0 : 16);
+            cp_async_16(smem_u32(Kd + jj * (D + 8) + e * 8), kc + (slot < 0 ? 0 : slot) * k_row + e * 8, slot < 0 ? 0 : 16);
             jj += k_djj, e += k_de;
             if (e >= ck) e -= ck, ++jj;
         }
         for (int jj = v_jj0, e = v_e0; jj < kKeys;) {
             const int64_t slot = slots[jj];
-            cp_async_16(smem_u32(Vd + jj * (DV + 8) + e * 8), vc + (slot < 0 ? 0 : slot) * DV + e * 8, slot < 0 ? 0 : 16);
+            cp_async_16(smem_u32(Vd + jj * (DV + 8) + e * 8), vc + (slot < 0 ? 0 : slot) * v_row + e * 8, slot < 0 ? 0 : 16);
             jj += v_djj, e += v_de;
             if (e >= cv) e -= cv, ++jj;
         }
@@ -221,7 +224,7 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
 #pragma unroll
             for (int n = 0; n < NT; ++n) sacc[n][0] = sacc[n][1] = sacc[n][2] = sacc[n][3] = 0.f;
 #pragma unroll
-            for (int kk = 0; kk < DMAX / 16; ++kk) {
+            for (int kk = 0; kk < DK / 16; ++kk) {
                 if (kk * 16 < D) {
 #pragma unroll
                     for (int np = 0; np < NT / 2; ++np) {
@@ -299,7 +302,7 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
                     }
                 if (__any_sync(0xffffffffu, corr[0] != 1.f || corr[1] != 1.f)) {   // no row's maximum moved: nothing to rescale
 #pragma unroll
-                    for (int n = 0; n < DMAX / 8; ++n) {
+                    for (int n = 0; n < DV_MAX / 8; ++n) {
                         o[n][0] *= corr[0];
                         o[n][1] *= corr[0];
                         o[n][2] *= corr[1];
@@ -315,7 +318,7 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
                 af[2] = pack2<__nv_bfloat16>(sacc[2 * kk + 1][0], sacc[2 * kk + 1][1]);
                 af[3] = pack2<__nv_bfloat16>(sacc[2 * kk + 1][2], sacc[2 * kk + 1][3]);
 #pragma unroll
-                for (int n2 = 0; n2 < DMAX / 16; ++n2) {
+                for (int n2 = 0; n2 < DV_MAX / 16; ++n2) {
                     if (n2 * 16 < DV) {
                         uint32_t r[4];
                         const __nv_bfloat16 *src = Vs + (key_off + kk * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * (DV + 8) + n2 * 16 + (lane >> 4) * 8;
@@ -337,7 +340,7 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
     }
 
     if constexpr (!ROWS_ARE_HEADS) {
-        __nv_bfloat16 *out = static_cast<__nv_bfloat16 *>(a.out) + (static_cast<int64_t>(tok0) * H + h0) * DV;
+        __nv_bfloat16 *out = static_cast<__nv_bfloat16 *>(a.out) + static_cast<int64_t>(tok0) * a.ld_out + h0 * DV;
         const __nv_bfloat16 *gate = a.gate ? static_cast<const __nv_bfloat16 *>(a.gate) + static_cast<int64_t>(tok0) * a.ld_gate + h0 * DV : nullptr;
 #pragma unroll
         for (int hf = 0; hf < 2; ++hf) {
@@ -345,7 +348,7 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
             if (row >= rows_w) continue;
             const float inv = SIG ? 1.f : 1.f / l_run[hf];
 #pragma unroll
-            for (int n = 0; n < DMAX / 8; ++n) {
+            for (int n = 0; n < DV_MAX / 8; ++n) {
                 if (n * 8 < DV) {
                     const int col = n * 8 + 2 * t4;
                     float v0 = o[n][2 * hf] * inv, v1 = o[n][2 * hf + 1] * inv;
@@ -354,7 +357,7 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
                         v0 *= sigmoidf_(gv.x);
                         v1 *= sigmoidf_(gv.y);
                     }
-                    *reinterpret_cast<uint32_t *>(out + static_cast<int64_t>(row) * H * DV + col) = pack2<__nv_bfloat16>(v0, v1);
+                    *reinterpret_cast<uint32_t *>(out + static_cast<int64_t>(row) * a.ld_out + col) = pack2<__nv_bfloat16>(v0, v1);
                 }
             }
         }
@@ -372,7 +375,7 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
                 l_s[warp * 16 + row] = l_run[hf];
             }
 #pragma unroll
-            for (int n = 0; n < DMAX / 8; ++n)
+            for (int n = 0; n < DV_MAX / 8; ++n)
                 if (n * 8 < DV) {
                     float *dst = o_s + (warp * 16 + row) * DV + n * 8 + 2 * t4;
                     dst[0] = o[n][2 * hf];
@@ -402,7 +405,7 @@ __global__ void __launch_bounds__(128, 3) softmax_attn_tc_kernel(const atoma_sof
             } else {
                 float v = SIG ? acc : acc / Lsum;
                 if (a.gate) v *= sigmoidf_(__bfloat162float(static_cast<const __nv_bfloat16 *>(a.gate)[static_cast<int64_t>(tok0) * a.ld_gate + h * DV + d]));
-                static_cast<__nv_bfloat16 *>(a.out)[(static_cast<int64_t>(tok0) * H + h) * DV + d] = __float2bfloat16_rn(v);
+                static_cast<__nv_bfloat16 *>(a.out)[static_cast<int64_t>(tok0) * a.ld_out + h * DV + d] = __float2bfloat16_rn(v);
             }
         }
     }
@@ -432,26 +435,33 @@ __global__ void __launch_bounds__(128) softmax_split_merge_kernel(const atoma_so
         }
         float v = acc / Lsum;
         if (a.gate) v *= sigmoidf_(__bfloat162float(static_cast<const __nv_bfloat16 *>(a.gate)[static_cast<int64_t>(t) * a.ld_gate + h * DV + d]));
-        static_cast<__nv_bfloat16 *>(a.out)[(static_cast<int64_t>(t) * H + h) * DV + d] = __float2bfloat16_rn(v);
+        static_cast<__nv_bfloat16 *>(a.out)[static_cast<int64_t>(t) * a.ld_out + h * DV + d] = __float2bfloat16_rn(v);
     }
 }
 
-template <int DMAX, bool ROWS_ARE_HEADS, bool EXACT, bool SIG>
+template <int DK, int DV_MAX, bool ROWS_ARE_HEADS, bool EXACT, bool SIG>
 cudaError_t launch_tc_exact(const atoma_softmax_attn_args &a, dim3 grid, size_t smem, int bias_n, int splits, float *partial, const float *head_bias,
                             cudaStream_t stream) {
     static int attr_dev = -1;
     const int dev = current_device_info().ordinal;
     if (attr_dev != dev) {
-        cudaFuncSetAttribute(softmax_attn_tc_kernel<DMAX, ROWS_ARE_HEADS, EXACT, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+        cudaFuncSetAttribute(softmax_attn_tc_kernel<DK, DV_MAX, ROWS_ARE_HEADS, EXACT, SIG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
         attr_dev = dev;
     }
-    return launch_ex(softmax_attn_tc_kernel<DMAX, ROWS_ARE_HEADS, EXACT, SIG>, grid, dim3(128), smem, stream, a, bias_n, splits, partial, head_bias);
+    return launch_ex(softmax_attn_tc_kernel<DK, DV_MAX, ROWS_ARE_HEADS, EXACT, SIG>, grid, dim3(128), smem, stream, a, bias_n, splits, partial, head_bias);
 }
-template <int DMAX, bool ROWS_ARE_HEADS, bool SIG>
+template <int DK, int DV_MAX, bool ROWS_ARE_HEADS, bool SIG>
+cudaError_t launch_tc_sized(const atoma_softmax_attn_args &a, dim3 grid, size_t smem, int bias_n, int splits, float *partial, const float *head_bias,
+                            cudaStream_t stream) {
+    return (a.dim == DK && a.vdim == DV_MAX) ? launch_tc_exact<DK, DV_MAX, ROWS_ARE_HEADS, true, SIG>(a, grid, smem, bias_n, splits, partial, head_bias, stream)
+                                             : launch_tc_exact<DK, DV_MAX, ROWS_ARE_HEADS, false, SIG>(a, grid, smem, bias_n, splits, partial, head_bias, stream);
+}
+template <bool ROWS_ARE_HEADS, bool SIG>
 cudaError_t launch_tc(const atoma_softmax_attn_args &a, dim3 grid, size_t smem, int bias_n, int splits, float *partial, const float *head_bias,
                       cudaStream_t stream) {
-    return (a.dim == DMAX && a.vdim == DMAX) ? launch_tc_exact<DMAX, ROWS_ARE_HEADS, true, SIG>(a, grid, smem, bias_n, splits, partial, head_bias, stream)
-                                             : launch_tc_exact<DMAX, ROWS_ARE_HEADS, false, SIG>(a, grid, smem, bias_n, splits, partial, head_bias, stream);
+    if (std::max(a.dim, a.vdim) <= 64) return launch_tc_sized<64, 64, ROWS_ARE_HEADS, SIG>(a, grid, smem, bias_n, splits, partial, head_bias, stream);
+    if (!SIG && a.dim <= 64) return launch_tc_sized<64, 128, ROWS_ARE_HEADS, false>(a, grid, smem, bias_n, splits, partial, head_bias, stream);   // long values
+    return launch_tc_sized<128, 128, ROWS_ARE_HEADS, SIG>(a, grid, smem, bias_n, splits, partial, head_bias, stream);
 }
 
 }  // namespace
@@ -463,7 +473,7 @@ bool attention_tc(const atoma_softmax_attn_args &a, const float *head_bias, cuda
     *taken = false;
     const int64_t kmax = std::max(a.dim, a.vdim);
     auto al = [](const void *p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
-    if (a.dtype != ATOMA_DTYPE_BF16 || a.max_query_len < 1 || !a.query_start || a.dim % 16 || a.vdim % 16 || kmax > 128 || !al(a.q) ||
+    if (a.dtype != ATOMA_DTYPE_BF16 || a.max_query_len < 1 || !a.query_start || a.dim % 16 || a.vdim % 16 || kmax > 128 || a.ld_out % 2 || !al(a.q) ||
         !al(a.k_cache) || !al(a.v_cache) || !al(a.out) || (a.gate && (!al(a.gate) || a.ld_gate % 8)) || current_device_info().cc_major < 9)
         return true;
     *taken = true;
@@ -488,8 +498,7 @@ bool attention_tc(const atoma_softmax_attn_args &a, const float *head_bias, cuda
             if (!partial) return false;
         }
         const dim3 grid(static_cast<unsigned>(splits), static_cast<unsigned>(a.B), static_cast<unsigned>(a.G * chunks));
-        const cudaError_t e = kmax <= 64 ? launch_tc<64, true, SIG>(a, grid, smem, 0, splits, partial, head_bias, stream)
-                                         : launch_tc<128, true, SIG>(a, grid, smem, 0, splits, partial, head_bias, stream);
+        const cudaError_t e = launch_tc<true, SIG>(a, grid, smem, 0, splits, partial, head_bias, stream);
         if (!hybrid::launched(e, "softmax_attn_tc_kernel<heads>")) return false;
         if (splits > 1 &&
             !hybrid::launched(launch_ex(softmax_split_merge_kernel, dim3(static_cast<unsigned>(a.B), static_cast<unsigned>(a.H)), dim3(128), 0, stream,
@@ -502,8 +511,7 @@ bool attention_tc(const atoma_softmax_attn_args &a, const float *head_bias, cuda
     const int bias_n = a.dist_bias ? static_cast<int>(std::min<int64_t>(a.dist_rows, kBiasSmem)) : 0;
     const TcLayout L = tc_layout(D, DV, bias_n);
     const dim3 grid(static_cast<unsigned>((a.max_query_len + kRowsCta - 1) / kRowsCta), static_cast<unsigned>(a.B), static_cast<unsigned>(a.H));
-    const cudaError_t e = kmax <= 64 ? launch_tc<64, false, SIG>(a, grid, L.total, bias_n, 1, nullptr, head_bias, stream)
-                                     : launch_tc<128, false, SIG>(a, grid, L.total, bias_n, 1, nullptr, head_bias, stream);
+    const cudaError_t e = launch_tc<false, SIG>(a, grid, L.total, bias_n, 1, nullptr, head_bias, stream);
     return hybrid::launched(e, "softmax_attn_tc_kernel<tokens>");
 }
 
@@ -537,6 +545,8 @@ bool hyb_sigmoid_attention_tc(const atoma_sigmoid_attn_args &s, cudaStream_t str
     a.dtype = s.dtype;
     a.max_query_len = s.max_query_len;
     a.max_seq_len = s.max_seq_len;
+    a.ld_out = s.H * s.vdim;
+    a.v_share = 1;
     return attention_tc<true>(a, s.head_bias, stream, taken);
 }
 

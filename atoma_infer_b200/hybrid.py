@@ -1,6 +1,6 @@
 """Hybrid (attention + recurrent) decoder models: description, device layout and the step executor's host side.
 
-A model family (atoma_infer_b200/lilovik.py, patadra.py, nemasun.py, surinex.py, mobunex.py) describes itself as a
+A model family (atoma_infer_b200/lilovik.py, patadra.py, nemasun.py, surinex.py, mobunex.py, lusalorn.py) describes itself as a
 `HybridSpec` — a list of layer RUNS, each a mixer (attention of some kind, a recurrence, or a pair of them) with its sizes and constants and an optional feed-forward (gated dense, or a mixture of experts) — and hands over its
 weights under the generic names below.  A design that runs a span of layers several times lists every run;
 runs that name the same `source` share one copy of the weights and have caches of their own.  `HybridExecutor` lays them out
@@ -45,6 +45,12 @@ Post-norm blocks (block_style "postnorm": x <- norm1(alpha x + mixer(x)), x <- n
   linear recurrent unit: w_y, w_x [S, width], b_y, b_x [S], tap_w [S, taps], tap_b [S], gate_r, gate_i [blocks, n, n] stored [out, in], gate_r_b,
                          gate_i_b [S], rate [S] (log of the decay at an open gate, <= 0), w_o [width, S]
   dense: w_gate_up [2 ff, width], w_down [width, ff]     experts: as for blocks on residual lanes
+  further for softmax attention: q_norm, k_norm [dim], b_o [width], differential attention (maps = 2): w_q [H 2 dim, width] and w_k
+                         [G 2 dim, width] with a head's two maps as neighbours, diff_lambda (a number)
+  sum of softmax attention and a state-space recurrence: the attention's tensors, and r_w_z, r_w_x [heads vdim, width], r_w_bc
+                         [2 groups state, width], r_w_dt [heads, width], r_tap_w [channels, taps], r_tap_b [channels] (channels x, B, C),
+                         r_dt_bias, r_a_log, r_skip [heads], r_norm [heads vdim], r_w_o [width, heads vdim]
+  without an embedding norm (embed_norm False) and with a pair-indexed table: pair_table [buckets + 1, width]
 The executor stacks the projections that read the same input into one matrix (rows padded to a multiple of 8).
 """
 from __future__ import annotations
@@ -63,7 +69,7 @@ from .ops import AtomaError
 from .scheduler import StepPlan
 from .worker import InputStager, SequenceInput
 
-MIXER_ATTENTION, MIXER_MINGRU, MIXER_LATENT, MIXER_SOFTMAX, MIXER_GLA, MIXER_PAIR, MIXER_LRU = 0, 1, 2, 3, 4, 5, 6
+MIXER_ATTENTION, MIXER_MINGRU, MIXER_LATENT, MIXER_SOFTMAX, MIXER_GLA, MIXER_PAIR, MIXER_LRU, MIXER_ATTENTION_SSM = 0, 1, 2, 3, 4, 5, 6, 7
 LONG_PORTION = 128        # tokens of a sequence in one step from which attention runs on the tensor-memory prefill kernel
                           # (latent attention: on expanded keys and values; softmax attention: on gathered ones)
 BLOCK_STYLES = {"sandwich": 0, "prenorm": 1, "lanes": 2, "parallel": 3, "postnorm": 4}
@@ -128,6 +134,13 @@ class SoftmaxAttentionSpec:
     distance_bias: bool = False    # weights carry dist_bias [rows, heads]
     bias: bool = False             # post-norm blocks: the projections have biases
     head_scale: bool = False       # post-norm blocks: a factor per head on the scores
+    # post-norm blocks, further: weighted q/k norms, rotary positions on q and k, a bias of the output projection
+    qk_norm: bool = False
+    rotary: Optional["RotarySpec"] = None
+    out_bias: bool = False
+    maps: int = 1                  # 2: differential attention, two softmax maps per head over the same values, combined as
+    diff: float = 0.0              #    (a1 - lambda a2) / rms(a1 - lambda a2) * (1 - diff), lambda from the weights
+    kv_from: Optional[int] = None  # the layer whose cached keys and values are used (no key and value projections of its own)
 
 
 @dataclass(frozen=True)
@@ -229,6 +242,44 @@ class LinearRecurrentSpec:
 
 
 @dataclass(frozen=True)
+class StateSpaceSpec:
+    """State-space recurrence: S <- exp(-exp(A_log) d) S + d B x^T, y = S^T C + D x per head with a step size d = softplus(. + dt_bias) per
+    head and token; x, B and C come through a short causal filter with silu, B and C are shared by groups of heads; y times silu(z) is
+    RMS-normed in `norm_groups` equal parts."""
+    heads: int
+    vdim: int
+    groups: int
+    state: int
+    norm_groups: int = 1
+    taps: int = 4
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def channels(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+
+@dataclass(frozen=True)
+class MixerSumSpec:
+    """Softmax attention and a state-space recurrence on the same input: left_scale * left + right_scale * right."""
+    left: SoftmaxAttentionSpec
+    right: StateSpaceSpec
+    left_scale: float = 1.0
+    right_scale: float = 1.0
+
+
+@dataclass(frozen=True)
+class PairTableSpec:
+    """A second embedding table looked up by (token before * mul_prev + token * mul_cur) mod buckets; its last row serves first tokens."""
+    buckets: int
+    mul_prev: int
+    mul_cur: int
+
+
+@dataclass(frozen=True)
 class ClampedMlpSpec:
     """Dense feed-forward W_down (g sigmoid(alpha g) (u + up_shift)) on g = min(W_gate h + b, limit), u = clamp(W_up h + b)."""
     ff: int
@@ -281,6 +332,13 @@ class LayerSpec:
     add_embedding: bool = False              # parallel blocks: the embedding rows are added to the stream before the layer
     pass_vector: Optional[int] = None        # ... and this row of weights["pass_vectors"]
     lru: Optional["LinearRecurrentSpec"] = None
+    mixer_sum: Optional["MixerSumSpec"] = None
+
+    @property
+    def own_kv(self) -> Optional[SoftmaxAttentionSpec]:
+        """The softmax attention whose keys and values this layer caches itself."""
+        a = self.mixer_sum.left if self.mixer_sum is not None else self.softmax
+        return a if a is not None and a.kv_from is None else None
 
 
 @dataclass(frozen=True)
@@ -302,15 +360,19 @@ class HybridSpec:
     embed_scale: float = 1.0                 # block_style "lanes": the embedding row times this (no position signal)
     residual_alpha: float = 1.0              # block_style "postnorm": the stream's factor in every sum
     depth_average: bool = False              # block_style "postnorm": a layer hands on a weighted sum of every result so far
+    embed_norm: bool = True                  # block_style "postnorm": the embedding rows are normed
+    branch_scale: Optional[float] = None     # block_style "postnorm": x <- alpha x + branch_scale norm(sublayer(x)) (None: the sum is normed)
+    pair_table: Optional[PairTableSpec] = None   # block_style "postnorm": a second embedding row per token
 
     @property
     def has_state(self) -> bool:
-        return any(l.mixer == "mingru" or l.taps > 1 or l.gla is not None or l.pair is not None or l.lru is not None for l in self.layers)
+        return any(l.mixer == "mingru" or l.taps > 1 or l.gla is not None or l.pair is not None or l.lru is not None or l.mixer_sum is not None
+                   for l in self.layers)
 
     def cache_bytes_per_token(self, dtype: torch.dtype) -> int:
         es = torch.empty((), dtype=dtype).element_size()
         return (sum(l.attention.kv_heads * (l.attention.dim + l.attention.vdim) * es for l in self.layers if l.mixer == "attention") +
-                sum(l.softmax.kv_heads * (l.softmax.dim + l.softmax.vdim) * es for l in self.layers if l.mixer == "softmax_attention") +
+                sum(a.kv_heads * (a.maps * a.dim + a.vdim) * es for a in (l.own_kv for l in self.layers) if a is not None) +
                 sum((l.latent.kv_rank + l.latent.rot_dim) * es for l in self.layers if l.mixer == "latent_attention") +
                 sum(l.pair.left.kv_heads * (l.pair.left.dim + l.pair.left.vdim) * es for l in self.layers if l.pair is not None))
 
@@ -466,10 +528,25 @@ class HybridExecutor:
             m.side_table, m.side_dim, m.side_table_width = self.side_table.data_ptr(), spec.side_dim, self.side_table.shape[1]
         m.lanes, m.embed_scale = spec.lanes, spec.embed_scale
         if spec.block_style == "postnorm":
-            self.embed_norm = small(weights["embed_norm"])
-            if tuple(self.embed_norm.shape) != (spec.width,) or tuple(self.final_norm.shape) != (spec.width,):
-                raise AtomaError(f"norms of the embedding and the output have shapes {tuple(self.embed_norm.shape)}, {tuple(self.final_norm.shape)}")
-            m.embed_norm, m.residual_alpha = self.embed_norm.data_ptr(), spec.residual_alpha
+            norms = {"final_norm": self.final_norm}
+            if spec.embed_norm:
+                norms["embed_norm"] = small(weights["embed_norm"])
+                m.embed_norm = norms["embed_norm"].data_ptr()
+            for name, t in norms.items():
+                if tuple(t.shape) != (spec.width,):
+                    raise AtomaError(f"{name} has shape {tuple(t.shape)}, the width is {spec.width}")
+            m.residual_alpha = spec.residual_alpha
+            if spec.branch_scale is not None:
+                m.norm_branch, m.branch_scale = 1, spec.branch_scale
+            if spec.pair_table is not None:
+                pt = spec.pair_table
+                table = big(weights["pair_table"])
+                if pt.buckets < 1 or tuple(table.shape) != (pt.buckets + 1, spec.width):
+                    raise AtomaError(f"pair table of shape {tuple(table.shape)} for {pt.buckets} buckets and a width of {spec.width}")
+                m.pair_table, m.pair_buckets = table.data_ptr(), pt.buckets
+                m.pair_mul_prev, m.pair_mul_cur = pt.mul_prev % pt.buckets, pt.mul_cur % pt.buckets
+        elif spec.pair_table is not None or spec.branch_scale is not None:
+            raise AtomaError("pair tables and normed branches are served by post-norm blocks")
         self._model = m
         self._stager = InputStager(device=dev, block_size=self.block_size, enable_chunked_prefill=True)
         self._extra_host = None
@@ -627,21 +704,13 @@ class HybridExecutor:
         L.norm1 = small(need("norm1", (W,))).data_ptr()
         if self.spec.depth_average:
             L.depth_w = small(need("depth_w", (i + 2,))).data_ptr()
+        L.mix_scale = 1.0
         if ls.mixer == "softmax_attention":
-            a = ls.softmax
-            if a.heads % a.kv_heads:
-                raise AtomaError(f"layer {i}: {a.kv_heads} kv heads do not divide {a.heads} heads")
-            if a.keep_first or a.values_are_keys or a.out_gate or a.distance_bias:
-                raise AtomaError(f"layer {i}: kept first tokens, values that are keys, output gates and distance tables are served on residual lanes")
             L.mixer = MIXER_SOFTMAX
-            L.heads, L.kv_heads, L.dim, L.vdim, L.scale, L.window = a.heads, a.kv_heads, a.dim, a.vdim, a.scale, a.window
-            bias = lambda name, n: need(name, (n,)) if a.bias else None
-            L.q_off = stack([need("w_q", (a.heads * a.dim, W))], bias("b_q", a.heads * a.dim))
-            L.k_off = stack([need("w_k", (a.kv_heads * a.dim, W))], bias("b_k", a.kv_heads * a.dim))
-            L.v_off = stack([need("w_v", (a.kv_heads * a.vdim, W))], bias("b_v", a.kv_heads * a.vdim))
-            if a.head_scale:
-                L.q_head_scale = small(need("head_scale", (a.heads,))).data_ptr()
-            L.w_o = big(need("w_o", (W, a.heads * a.vdim))).data_ptr()
+            self._place_postnorm_softmax(L, i, ls.softmax, w, need, stack, small)
+            L.w_o = big(need("w_o", (W, ls.softmax.heads * ls.softmax.vdim))).data_ptr()
+        elif ls.mixer == "attention_ssm":
+            self._place_mixer_sum(L, i, ls.mixer_sum, w, need, stack, big, small)
         elif ls.mixer == "latent_attention":
             a = ls.latent
             if a.sink:
@@ -686,7 +755,7 @@ class HybridExecutor:
             L.lru_rate = small(need("rate", (d.width,))).data_ptr()
             L.w_o = big(need("w_o", (W, d.width))).data_ptr()
         else:
-            raise AtomaError(f"layer {i}: post-norm blocks take the mixers softmax_attention, latent_attention and lru, not {ls.mixer!r}")
+            raise AtomaError(f"layer {i}: post-norm blocks take the mixers softmax_attention, attention_ssm, latent_attention and lru, not {ls.mixer!r}")
         L.w_qkv, L.b_qkv = big(torch.cat(parts, 0)).data_ptr(), small(torch.cat(biases, 0)).data_ptr()
         L.proj_cols = sum(p.shape[0] for p in parts)
         L.has_mlp = 1 if ls.mlp is not None or ls.moe is not None else 0
@@ -703,6 +772,88 @@ class HybridExecutor:
         if e.identity or e.shared_limit or e.shared_gate:
             raise AtomaError(f"layer {i}: identity experts and clamped or gated shared experts are served by other block styles")
         self._place_routed(L, i, e, w, big, small)
+
+    def _place_postnorm_softmax(self, L, i: int, a: SoftmaxAttentionSpec, w: dict, need, stack, small) -> None:
+        """Softmax attention of a post-norm layer.  Differential attention runs as attention of twice the heads: a group's query heads under
+        the first map, then under the second, on a key head of their own, and both key heads share the group's value head."""
+        W = self.spec.width
+        if a.heads % a.kv_heads:
+            raise AtomaError(f"layer {i}: {a.kv_heads} kv heads do not divide {a.heads} heads")
+        if a.keep_first or a.values_are_keys or a.out_gate or a.distance_bias:
+            raise AtomaError(f"layer {i}: kept first tokens, values that are keys, output gates and distance tables are served on residual lanes")
+        if a.maps not in (1, 2):
+            raise AtomaError(f"layer {i}: {a.maps} softmax maps per head (1 or 2 are supported)")
+        H, G, M = a.heads, a.kv_heads, a.maps
+        L.heads, L.kv_heads, L.dim, L.vdim, L.scale, L.window, L.v_share = M * H, M * G, a.dim, a.vdim, a.scale, a.window, M
+
+        def by_map(t):       # query rows [H][maps][dim] -> [G][maps][H / G][dim]
+            return t if M == 1 else t.reshape(G, H // G, M, a.dim, -1).transpose(1, 2).reshape(t.shape).contiguous()
+
+        def bias(name, n):
+            return need(name, (n,)) if a.bias else None
+
+        bq = bias("b_q", M * H * a.dim)
+        L.q_off = stack([by_map(need("w_q", (M * H * a.dim, W)))], None if bq is None else by_map(bq))
+        if a.kv_from is None:
+            L.k_off = stack([need("w_k", (M * G * a.dim, W))], bias("b_k", M * G * a.dim))
+            L.v_off = stack([need("w_v", (G * a.vdim, W))], bias("b_v", G * a.vdim))
+        else:
+            self._kv_source(i, a)
+            L.k_off = L.v_off = -1
+        if a.qk_norm:
+            L.q_norm = small(need("q_norm", (a.dim,))).data_ptr()
+            L.k_norm = small(need("k_norm", (a.dim,))).data_ptr() if a.kv_from is None else None
+        if a.head_scale:
+            hs = need("head_scale", (H,))
+            L.q_head_scale = small(hs.reshape(G, H // G).repeat_interleave(M, 0).reshape(-1)).data_ptr()
+        if a.rotary is not None:
+            self._place_rotation(L, i, a.rotary, a.dim, small)
+        if a.out_bias:
+            L.b_o = small(need("b_o", (W,))).data_ptr()
+        if M == 2:
+            L.diff_lambda, L.diff_gain = float(w["diff_lambda"]), 1.0 - a.diff
+            if L.diff_gain == 0.0:
+                raise AtomaError(f"layer {i}: a difference weight of one leaves nothing of the result")
+
+    def _kv_source(self, i: int, a: SoftmaxAttentionSpec) -> int:
+        """The layer whose caches layer i reads."""
+        j = a.kv_from
+        src = self.spec.layers[j].softmax if 0 <= j < i else None
+        if src is None or src.kv_from is not None or (src.kv_heads, src.maps, src.dim, src.vdim) != (a.kv_heads, a.maps, a.dim, a.vdim):
+            raise AtomaError(f"layer {i}: keys and values of layer {j}, which is no earlier softmax-attention layer with projections of its own and "
+                             f"the same key and value heads")
+        return j
+
+    def _place_mixer_sum(self, L, i: int, ms: MixerSumSpec, w: dict, need, stack, big, small) -> None:
+        """Softmax attention beside a state-space recurrence.  Both results are columns of ONE row that one output projection reads; the
+        scales are kept out of the 16-bit matrices: the sum is left_scale (left + right_scale / left_scale right), the inner factor
+        goes into the (float32) norm weight of the recurrence and the outer one into the residual update."""
+        W, a, d = self.spec.width, ms.left, ms.right
+        if a.maps != 1 or a.out_bias or a.kv_from is not None:
+            raise AtomaError(f"layer {i}: the attention of a summed layer has one map, no output bias and a cache of its own")
+        if d.groups < 1 or d.heads % d.groups or d.norm_groups < 1 or d.inner % d.norm_groups:
+            raise AtomaError(f"layer {i}: {d.heads} heads in {d.groups} groups, {d.inner} channels in {d.norm_groups} norm groups")
+        if not 1 <= d.taps <= 16:
+            raise AtomaError(f"layer {i}: {d.taps} taps of the short filter (1 to 16 are supported)")
+        self._place_postnorm_softmax(L, i, a, w, need, stack, small)
+        L.mixer = MIXER_ATTENTION_SSM
+        L.rg_off = stack([need("r_w_z", (d.inner, W))])
+        L.rv_off = stack([need("r_w_x", (d.inner, W)), need("r_w_bc", (2 * d.groups * d.state, W))])
+        L.ra_off = stack([need("r_w_dt", (d.heads, W))])
+        L.r_heads, L.r_kv_heads, L.r_dim, L.r_vdim, L.r_taps, L.r_norm_groups = d.heads, d.groups, d.state, d.vdim, d.taps, d.norm_groups
+        L.r_tap_w, L.r_tap_bias = small(need("r_tap_w", (d.channels, d.taps))).data_ptr(), small(need("r_tap_b", (d.channels,))).data_ptr()
+        L.r_dt_bias, L.r_a_log, L.r_skip = (small(need(k, (d.heads,))).data_ptr() for k in ("r_dt_bias", "r_a_log", "r_skip"))
+        w_left = need("w_o", (W, a.heads * a.vdim))
+        outer, inner = (ms.left_scale, ms.right_scale / ms.left_scale) if ms.left_scale != 0.0 else (1.0, ms.right_scale)
+        if ms.left_scale == 0.0:
+            w_left = torch.zeros_like(w_left)
+        L.mix_scale = outer
+        L.r_head_norm = small(need("r_norm", (d.inner,)).double() * inner).data_ptr()
+        gap = torch.zeros((W, -w_left.shape[1] % 8), dtype=w_left.dtype, device=w_left.device)
+        tail = torch.zeros((W, -d.inner % 8), dtype=w_left.dtype, device=w_left.device)
+        L.r_mix_off = w_left.shape[1] + gap.shape[1]
+        L.mix_cols = L.r_mix_off + d.inner + tail.shape[1]
+        L.w_o = big(torch.cat([w_left, gap, need("r_w_o", (W, d.inner)).to(w_left.device), tail], 1)).data_ptr()
 
     def _place_parallel(self, L, i: int, ls: LayerSpec, w: dict, big, small) -> None:
         """Device copies and sizes of one parallel layer: the projections that read the mixer's input stacked into one matrix
@@ -833,6 +984,9 @@ class HybridExecutor:
             n += max(0, d.taps - 1) * (2 * d.kv_heads * d.dim + d.heads * d.vdim) + d.heads * d.dim * d.vdim
         if ls.lru is not None:
             n += max(0, ls.lru.taps - 1) * ls.lru.width + ls.lru.width
+        if ls.mixer_sum is not None:
+            d = ls.mixer_sum.right
+            n += max(0, d.taps - 1) * d.channels + d.heads * d.state * d.vdim
         return n
 
     def _run_state(self, L, i: int, ls: LayerSpec, weights: dict, small, rows: int) -> None:
@@ -842,9 +996,12 @@ class HybridExecutor:
         if ls.mixer == "latent_attention":
             lc = torch.zeros((rows, ls.latent.kv_rank + ls.latent.rot_dim), dtype=dtype, device=dev)
             L.latent_cache = lc.data_ptr()
-        elif ls.mixer in ("pair", "softmax_attention"):
-            a = ls.pair.left if ls.pair is not None else ls.softmax
-            kc = torch.zeros((rows, a.kv_heads, a.dim), dtype=dtype, device=dev)
+        elif ls.softmax is not None and ls.softmax.kv_from is not None:
+            kc, vc = self.k_caches[ls.softmax.kv_from], self.v_caches[ls.softmax.kv_from]
+            L.k_cache, L.v_cache = kc.data_ptr(), vc.data_ptr()
+        elif ls.mixer in ("pair", "softmax_attention", "attention_ssm"):
+            a = ls.pair.left if ls.pair is not None else ls.own_kv
+            kc = torch.zeros((rows, getattr(a, "maps", 1) * a.kv_heads, a.dim), dtype=dtype, device=dev)
             vc = torch.zeros((rows, a.kv_heads, a.vdim), dtype=dtype, device=dev)
             L.k_cache, L.v_cache = kc.data_ptr(), vc.data_ptr()
         n = self.state_floats(ls)
@@ -879,8 +1036,8 @@ class HybridExecutor:
             self._logits = torch.empty((cap, self.spec.vocab), dtype=torch.float32, device=self.device)
             self._next = torch.zeros((cap,), dtype=torch.int32, device=self.device)
 
-    def _extras(self, token_seq: np.ndarray, state_slots: np.ndarray, selected: np.ndarray):
-        n = token_seq.size + state_slots.size + selected.size
+    def _extras(self, token_seq: np.ndarray, state_slots: np.ndarray, prev_tokens: np.ndarray, selected: np.ndarray):
+        n = token_seq.size + state_slots.size + prev_tokens.size + selected.size
         if self._extra_host is None or self._extra_host.numel() < n:
             cap = 1 << max(10, (n - 1).bit_length())
             torch.cuda.synchronize(self.device)
@@ -890,17 +1047,18 @@ class HybridExecutor:
             torch.cuda.current_stream(self.device).synchronize()   # the previous copy has read the pinned buffer
         h = self._extra_host.numpy()
         a, b = token_seq.size, token_seq.size + state_slots.size
-        h[:a], h[a:b], h[b:n] = token_seq, state_slots, selected
+        c = b + prev_tokens.size
+        h[:a], h[a:b], h[b:c], h[c:n] = token_seq, state_slots, prev_tokens, selected
         self._extra_dev[:n].copy_(self._extra_host[:n], non_blocking=True)
         d = self._extra_dev
-        return d[:a], d[a:b], d[b:n]
+        return d[:a], d[a:b], d[b:c], d[c:n]
 
     # ---- one step ----
     def execute(self, plan: StepPlan, want_residual_trace: bool = False) -> StepOutput:
         chunks = plan.chunks
         if not chunks:
             return StepOutput(None, None)
-        seqs, token_seq, slots, selected, rows = [], [], [], [], []
+        seqs, token_seq, slots, prev, selected, rows = [], [], [], [], [], []
         t0 = 0
         for b, c in enumerate(chunks):
             end = c.start + c.count
@@ -915,6 +1073,7 @@ class HybridExecutor:
                                       is_prompt=True))
             token_seq.append(np.full(c.count, b, dtype=np.int32))
             slots.append(0 if c.state_slot is None else c.state_slot)
+            prev.append(int(c.seq.tokens[c.start - 1]) if c.start > 0 else -1)
             for w in c.want:
                 if not 0 <= w < c.count:
                     raise AtomaError(f"sequence {c.seq.seq_id}: wanted offset {w} outside a chunk of {c.count}")
@@ -925,8 +1084,8 @@ class HybridExecutor:
         lay, v = self._stager.prepare_raw(seqs)
         if lay.num_tokens != T or lay.num_slots != T:
             raise AtomaError(f"step inputs: {lay.num_tokens} tokens / {lay.num_slots} slots prepared for a plan of {T}")
-        tseq, sslots, sel = self._extras(np.concatenate(token_seq), np.asarray(slots, dtype=np.int32),
-                                         np.asarray(selected, dtype=np.int32))
+        tseq, sslots, before, sel = self._extras(np.concatenate(token_seq), np.asarray(slots, dtype=np.int32), np.asarray(prev, dtype=np.int32),
+                                                 np.asarray(selected, dtype=np.int32))
         self._reserve(T, S)
         bt = v["block_tables"]
         trace = (torch.empty((len(self.spec.layers), T, self.spec.width), dtype=torch.float32, device=self.device)
@@ -942,6 +1101,7 @@ class HybridExecutor:
         hb.tokens, hb.positions, hb.slot_mapping = v["tokens"].data_ptr(), v["positions"].data_ptr(), v["slot_mapping"].data_ptr()
         hb.token_seq, hb.query_start, hb.context_lens = tseq.data_ptr(), v["query_start"].data_ptr(), v["context_lengths"].data_ptr()
         hb.block_tables, hb.state_slots = bt.data_ptr(), sslots.data_ptr()
+        hb.prev_tokens = before.data_ptr()
         hb.selected = sel.data_ptr() if S else None
         hb.scratch, hb.scratch_bytes = self._scratch.data_ptr(), self._scratch.numel()
         hb.logits = self._logits.data_ptr() if S else None
@@ -953,7 +1113,7 @@ class HybridExecutor:
         if L.atoma_last_status() != 0:
             raise AtomaError(L.atoma_last_error().decode())
         self.launches_last_step = int(L.atoma_launch_count())
-        self._last = (hb, tseq, sslots, sel, trace)
+        self._last = (hb, tseq, sslots, before, sel, trace)
         return StepOutput(self._logits[:S] if S else None, self._next[:S] if S else None, rows, trace)
 
 

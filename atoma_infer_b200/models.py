@@ -99,6 +99,18 @@ def _mobunex_needs_state(cfg) -> bool:
     return any(l["type"] == "rglru" for l in cfg["layers"])
 
 
+def _build_lusalorn(cfg, ckpt, dtype, device, cache: CacheConfig):
+    from . import lusalorn
+    from .hybrid import HybridExecutor
+    spec = lusalorn.spec_from_config(cfg)
+    weights = lusalorn.weights_from_checkpoint(spec, ckpt)
+    return HybridExecutor(spec, weights, dtype, device, cache.num_blocks, cache.block_size, cache.num_state_slots)
+
+
+def _lusalorn_needs_state(cfg) -> bool:
+    return any(l["type"] == "parallel" for l in cfg["layers"])
+
+
 def _build_llama(cfg, ckpt, dtype, device, cache: CacheConfig):
     from .llama_engine import LlamaExecutor
     return LlamaExecutor.from_checkpoint(cfg, ckpt, dtype, device, cache)
@@ -109,4 +121,5 @@ register_model("Patadra", _build_patadra)
 register_model("Nemasun", _build_nemasun)
 register_model("Surinex", _build_surinex, lambda cfg: True)       # input histories of the tap filters, in every layer
 register_model("Mobunex", _build_mobunex, _mobunex_needs_state)
+register_model("Lusalorn", _build_lusalorn, _lusalorn_needs_state)
 register_model("LlamaForCausalLM", _build_llama)

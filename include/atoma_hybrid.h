@@ -47,6 +47,13 @@
  * sliding window with a sigmoid gate on the heads' outputs, and a mixture of experts whose groups are ranked by the sum of their two
  * best choice scores.
  *
+ * The sixth design is Lusalorn: blocks that norm the sublayer's RESULT only (x <- x + m norm(sublayer(x)), the sublayer reads the stream
+ * itself), an embedding with a second row looked up by a hash of the pair (token before, token), differential attention (two softmax
+ * maps per head over the same values, combined as a1 - lambda a2 at unit root mean square) under a sliding window with projection
+ * biases, layers that read an earlier layer's cached keys and values, and a SUM of two mixers on the same input: softmax attention with
+ * rotary positions (YaRN-scaled) beside a state-space recurrence (short causal filter, a scalar decay and a step size per head and
+ * token, keys and queries shared by groups of heads, a skip term, a gate before a grouped norm).
+ *
  * Conventions: row-major; `dtype` is the number format of activations, large weights and the caches:
  * 1 = bfloat16, 2 = float32 (true 32-bit arithmetic: no reduced-precision matrix mode).  Whatever the
  * dtype, the residual stream, norm statistics, attention scores and weights, recurrent state and all
@@ -390,11 +397,21 @@ typedef struct atoma_softmax_attn_args {
      * the sum of their tokens and of their contexts.  bfloat16 heads of 64 or 128 with dim = vdim run them on the tensor-memory
      * prefill kernel: the keys and values their queries can see through the window are gathered from the pages, the distance
      * term is added inside that kernel's softmax, the kept first tokens behind the window are a second short pass merged through
-     * the log-sum-exp, and the gate is applied in the merge. */
+     * the log-sum-exp, and the gate is applied in the merge.  Without a table, kept tokens and a gate, dim and vdim may differ (vdim 64
+     * or 128, dim a multiple of 8 up to vdim + 64). */
     int32_t long_min_q, long_seqs;
     int64_t long_tokens, long_ctx_sum;
+    int64_t ld_out;               /* row stride of out (0: H vdim) */
+    int64_t v_share;              /* neighbouring key heads that share one value head (0: 1): the value cache has G / v_share heads per row */
 } atoma_softmax_attn_args;
 void atoma_softmax_attention_paged(const atoma_softmax_attn_args *args, atoma_stream_t stream);
+
+/* Two softmax maps per head into one result.  maps [T, 2 H vdim] (`dtype`) holds the heads' outputs by groups of rep = H / G query heads:
+ * group g's rep outputs under the first map, then its rep outputs under the second.  Per token and head h = g rep + r, in float32:
+ *   o = a1 - lambda a2;   out[t, h vdim ..] = o / sqrt(mean(o^2) + eps) * gain
+ * out [T, H vdim] in `dtype`. */
+void atoma_differential_combine(const void *maps, void *out, int64_t T, int64_t H, int64_t G, int64_t vdim, float lambda, float gain,
+                                float eps, uint32_t dtype, atoma_stream_t stream);
 
 /* Router with a restricted choice, float32.  z = w_router h over `outputs` router rows (experts, then identity experts);
  * s = softmax(z) (score_fn 1) or sigmoid(z) (0); choice score c = s + correction (NULL: none).  The outputs form `groups`
@@ -486,6 +503,8 @@ void atoma_tap_filter(const atoma_tap_filter_args *args, atoma_stream_t stream);
  *     q, k <- x / sqrt(sum(x^2) + unit_eps) (q also times q_scale);  beta = sigmoid(b_pre);
  *     g = exp(-exp(a_log[h]) * softplus(a_pre + dt_bias[h]));
  *     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+ *   kind 2, state-space recurrence (q, k [T, G dim] shared by H / G heads, v [T, H vdim]; per head a_pre [T, H]):
+ *     d = softplus(a_pre + dt_bias[h]);  S <- exp(-exp(a_log[h]) d) S + d k v^T;  o = S^T q * q_scale + skip[h] v
  * q, k, v, z, b_pre, a_pre are columns of `dtype` matrices with their own row strides; out float32 [T, H vdim].
  */
 typedef struct atoma_state_scan_args {
@@ -493,7 +512,7 @@ typedef struct atoma_state_scan_args {
     const void *q, *k, *v, *z, *b_pre, *a_pre;
     int64_t ld_q, ld_k, ld_v, ld_z, ld_b, ld_a;
     const float *z_bias;          /* [H dim] (kind 0) */
-    const float *a_log, *dt_bias; /* [H] (kind 1) */
+    const float *a_log, *dt_bias; /* [H] (kinds 1, 2) */
     float tau, q_scale, unit_eps;
     float *state;
     int64_t state_stride;
@@ -501,6 +520,7 @@ typedef struct atoma_state_scan_args {
     float *out;
     int64_t T, B, H, G, dim, vdim;
     uint32_t dtype;
+    const float *skip;            /* [H] or NULL (kind 2) */
 } atoma_state_scan_args;
 void atoma_state_scan(const atoma_state_scan_args *args, atoma_stream_t stream);
 
@@ -509,6 +529,13 @@ void atoma_state_scan(const atoma_state_scan_args *args, atoma_stream_t stream);
 void atoma_headnorm_gate(const float *o, const float *weight, const void *gate, int64_t ld_gate, void *out, int64_t T, int64_t H,
                          int64_t vdim, float eps, uint32_t dtype, atoma_stream_t stream);
 
+/* A recurrence's read-out through its gate, then normed: u = o[t, :] * silu(gate[t, :]);
+ *   out[t, c] = u[c] / sqrt(mean over c's part of u^2 + eps) * weight[c]        (`parts` equal consecutive parts of the n columns)
+ * o float32 [T, n], gate (row stride ld_gate) and out (row stride ld_out) in `dtype`.  The zero_before columns in front of out's and the
+ * zero_after columns behind them are set to zero (padding between the parts of a wider row). */
+void atoma_gate_groupnorm(const float *o, const void *gate, int64_t ld_gate, const float *weight, void *out, int64_t ld_out, int64_t T,
+                          int64_t n, int64_t parts, int64_t zero_before, int64_t zero_after, float eps, uint32_t dtype, atoma_stream_t stream);
+
 /*
  * After a fused projection proj[t, :] (row stride ld): queries at q_off (H heads of dim), keys at k_off (G of dim), values
  * at v_off (G of vdim).  Per head: RMS norm over dim with q_weight / k_weight ([dim], NULL: none), then the first
@@ -516,6 +543,9 @@ void atoma_headnorm_gate(const float *o, const float *weight, const void *gate, 
  * (i, i + rot_pairs) (0); the values' first 2 v_pairs entries likewise by v_freq (v_freq NULL: stored as projected).
  * bias (float32, indexed by the columns of proj; NULL: none) is added to the projections first; unit_norm 1 divides every query
  * and key head by its root mean square also without a weight; q_head_scale [H] (NULL: none) multiplies a normed query head.
+ * The q / k angles are formed to twice float32's precision: qk_freq_lo is what float32 drops of the frequencies (NULL: nothing);
+ * cos and sin are scaled by qk_amplitude (0: 1).  v_heads: value heads when there are fewer than key heads (0: G).
+ * slot_mapping NULL: queries only.
  * q -> q_out [T, H dim]; k, v -> cache rows slot_mapping[t] (slot < 0 is skipped).
  */
 typedef struct atoma_qkv_rope_args {
@@ -532,6 +562,9 @@ typedef struct atoma_qkv_rope_args {
     uint32_t dtype;
     const float *bias, *q_head_scale;
     int32_t unit_norm;
+    const float *qk_freq_lo;
+    float qk_amplitude;
+    int64_t v_heads;
 } atoma_qkv_rope_args;
 void atoma_qkv_headnorm_rope_cache(const atoma_qkv_rope_args *args, atoma_stream_t stream);
 
@@ -568,6 +601,15 @@ void atoma_latent_expand_values(const float *o_lat, const void *w_uv, const void
 /* Post-norm blocks with a depth average; real-gated linear recurrent unit                      */
 /* ------------------------------------------------------------------------------------------ */
 
+/* Embedding rows with a second table looked up by the pair (token before, token), for a mixed batch:
+ *   x[t, :] = table[tokens[t], :] + pair_table[row, :],  row = (before * mul_prev + tokens[t] * mul_cur) mod buckets   (64-bit integers)
+ * and row = buckets for a sequence's first token.  `before` is tokens[t - 1] inside a sequence's portion and prev_tokens[b] (negative: the
+ * portion starts the sequence) at its first token.  pair_table [buckets + 1, width] (NULL: x is the plain row).  x float32;
+ * h [T, width] (NULL: not written) = x in `dtype`. */
+void atoma_embed_pairs(const uint32_t *tokens, const int32_t *token_seq, const int32_t *query_start, const int32_t *prev_tokens, const void *table,
+                       const void *pair_table, int64_t buckets, int64_t mul_prev, int64_t mul_cur, float *x, void *h, int64_t T, int64_t width,
+                       int64_t vocab, uint32_t dtype, atoma_stream_t stream);
+
 /*
  * Residual update of a post-norm block, fused with the sum of the token's expert rows and the average over depth.  Per token t:
  *   v = alpha * x[t, :] + (y ? y[t, :] : 0) + sum_{k < top} (top_expert[t, k] >= 0: expert_out[pair_row[t top + k], :])
@@ -575,6 +617,9 @@ void atoma_latent_expand_values(const float *o_lat, const void *w_uv, const void
  *   x[t, :] = n                                                              (depth_n = 0)
  *   depth[depth_n - 1][t, :] = n;  x[t, :] = sum_{j < depth_n} depth_w[j] depth[j][t, :]   (depth_n > 0; depth_w NULL: x = n)
  *   h[t, :] = x[t, :] in `dtype` (NULL: not written);   trace[t, :] = x[t, :] (NULL: not written)
+ * norm_branch = 1 norms the sublayer's result instead of the sum:
+ *   v = y_scale * y[t, :] + y_bias + expert rows;   n = alpha * x[t, :] + branch_scale * v / sqrt(mean(v^2) + eps) * (weight_offset + w_norm)
+ * (y_bias NULL: none; y_scale and branch_scale are used in this form only).
  * x float32 [T, width] in place; depth float32 [.., T, width] (row j of the average at j T width), rows 0 .. depth_n - 2 written by
  * earlier calls.  y, expert_out, h in `dtype`.  Experts' rows are added in the order of k, depth rows in the order of j.
  */
@@ -594,6 +639,9 @@ typedef struct atoma_postnorm_args {
     int64_t T, width;
     float alpha, eps, weight_offset;
     uint32_t dtype;
+    int32_t norm_branch;
+    const float *y_bias;          /* [width] or NULL */
+    float y_scale, branch_scale;
 } atoma_postnorm_args;
 void atoma_postnorm_residual(const atoma_postnorm_args *args, atoma_stream_t stream);
 
@@ -641,7 +689,7 @@ void atoma_linear_scan(const atoma_linear_scan_args *args, atoma_stream_t stream
 /* Step executor                                                                                */
 /* ------------------------------------------------------------------------------------------ */
 enum { ATOMA_MIXER_SIGMOID_ATTENTION = 0, ATOMA_MIXER_MINGRU = 1, ATOMA_MIXER_LATENT_ATTENTION = 2, ATOMA_MIXER_SOFTMAX_ATTENTION = 3,
-       ATOMA_MIXER_GLA = 4, ATOMA_MIXER_PAIR = 5, ATOMA_MIXER_LRU = 6 };
+       ATOMA_MIXER_GLA = 4, ATOMA_MIXER_PAIR = 5, ATOMA_MIXER_LRU = 6, ATOMA_MIXER_ATTENTION_SSM = 7 };
 enum { ATOMA_BLOCK_SANDWICH = 0, ATOMA_BLOCK_PRENORM = 1, ATOMA_BLOCK_LANES = 2, ATOMA_BLOCK_PARALLEL = 3,
        ATOMA_BLOCK_POSTNORM = 4 };
 enum { ATOMA_SCORE_SIGMOID = 0, ATOMA_SCORE_SOFTMAX = 1 };
@@ -750,6 +798,20 @@ typedef struct atoma_hybrid_layer {
     const void *lru_w;               /* [lru_blocks, 2 n, n] */
     const float *lru_bias_r, *lru_bias_i, *lru_rate, *r_tap_bias; /* [lru_width] */
     const void *w_uk_rot;            /* [heads (dim + rot_dim), kv_rank + rot_dim]: a cached row -> the heads' whole keys, or NULL */
+    /* softmax attention, further: bias of the output projection [width] or NULL (joined in the residual update); v_share key heads per
+     * value head (0: 1); v_off < 0: no key and value projections, the caches are an earlier layer's; diff_gain != 0: differential, `heads`
+     * counts both maps' heads (laid out by groups, first map then second), w_o reads heads / 2 of them */
+    const float *b_o;
+    int64_t v_share;
+    float diff_lambda, diff_gain;
+    /* sum of softmax attention and a state-space recurrence on the same input: attention as above; recurrence of r_heads heads of r_vdim,
+     * r_kv_heads groups of r_dim states, filter [r_heads r_vdim + 2 r_kv_heads r_dim, r_taps] with r_tap_bias over the columns [x | B | C] at
+     * rv_off, gate at rg_off, step sizes at ra_off, r_a_log, r_dt_bias, r_skip [r_heads], norm weight r_head_norm [r_heads r_vdim] in
+     * r_norm_groups parts.  w_o [width, mix_cols] reads [attention | padding | recurrence at column r_mix_off | padding] in one product; the sum
+     * is its result times mix_scale.  The layer's state row = [filter history | r_heads r_dim r_vdim] */
+    const float *r_skip;
+    int64_t r_norm_groups, mix_cols, r_mix_off;
+    float mix_scale;
 } atoma_hybrid_layer;
 
 typedef struct atoma_hybrid_model {
@@ -775,6 +837,11 @@ typedef struct atoma_hybrid_model {
     /* ---- post-norm designs ---- */
     const float *embed_norm; /* [width]: norm of the embedding rows */
     float residual_alpha;   /* the stream's factor in every sum */
+    /* embed_norm NULL: the embedding rows as they are; norm_branch 1: the sublayers' results are normed and added times branch_scale */
+    float branch_scale;
+    int32_t norm_branch;
+    const void *pair_table; /* [pair_buckets + 1, width] second embedding table (atoma_embed_pairs) or NULL */
+    int64_t pair_buckets, pair_mul_prev, pair_mul_cur;
 } atoma_hybrid_model;
 
 typedef struct atoma_hybrid_batch {
@@ -798,6 +865,7 @@ typedef struct atoma_hybrid_batch {
      * there are, the sum of their tokens and of their contexts (tokens already cached) */
     int32_t long_seqs, long_min_q;
     int64_t long_tokens, long_ctx_sum;
+    const int32_t *prev_tokens;   /* [B] token before the portion, -1 at a sequence's start (models with a pair table; else may be NULL) */
 } atoma_hybrid_batch;
 
 int64_t atoma_hybrid_abi_sizeof(int which); /* 0 layer, 1 model, 2 batch, 3 attention args, 4 gated residual args, 5 latent attention args, 6 expert args, 7 expanded attention args, 8 lanes update args, 9 softmax attention args, 10 parallel residual args, 11 tap filter args, 12 state scan args, 13 rotary cache args, 14 post-norm args, 15 gate args, 16 linear scan args */
