@@ -352,9 +352,11 @@ def qk_headnorm_cache(proj, q_off, k_off, v_off, q_w, k_w, offset, slots, k_cach
 
 
 def softmax_attention_paged(q, k_cache, v_cache, positions, token_seq, block_tables, H, G, dim, vdim, block_size, scale, window=0,
-                            keep_first=0, dist_bias=None, gate=None, max_query_len=None, query_start=None, max_seq_len=None, long_min_q=0, long_stats=None):
+                            keep_first=0, dist_bias=None, gate=None, max_query_len=None, query_start=None, max_seq_len=None, long_min_q=0, long_stats=None,
+                            out=None, v_share=1):
     """long_min_q > 0: sequences with at least that many tokens in the step take the long-portion path (where the shapes allow);
-    long_stats = (how many such sequences, the sum of their tokens, the sum of their contexts) saves the host reads that find them."""
+    long_stats = (how many such sequences, the sum of their tokens, the sum of their contexts) saves the host reads that find them.
+    out: a [T, >= H vdim] view with a row stride of its own; v_share neighbouring key heads share one value head."""
     from ._lib import SoftmaxAttnArgs
     T = q.shape[0]
     if query_start is None:
@@ -364,7 +366,8 @@ def softmax_attention_paged(q, k_cache, v_cache, positions, token_seq, block_tab
         max_query_len = int((query_start[1:] - query_start[:-1]).max())
     if max_seq_len is None:
         max_seq_len = int(positions.max()) + 1
-    out = torch.empty((T, H * vdim), dtype=q.dtype, device=q.device)
+    if out is None:
+        out = torch.empty((T, H * vdim), dtype=q.dtype, device=q.device)
     a = SoftmaxAttnArgs()
     a.q, a.k_cache, a.v_cache, a.out, a.gate = _p(q), _p(k_cache), _p(v_cache), _p(out), _p(gate)
     a.ld_gate = gate.stride(0) if gate is not None else 0
@@ -373,6 +376,7 @@ def softmax_attention_paged(q, k_cache, v_cache, positions, token_seq, block_tab
     a.T, a.B, a.max_blocks, a.H, a.G, a.dim, a.vdim = T, block_tables.shape[0], block_tables.shape[1], H, G, dim, vdim
     a.block_size, a.window, a.keep_first, a.scale, a.dtype = block_size, window, keep_first, scale, _CODES[q.dtype]
     a.max_query_len, a.max_seq_len = int(max_query_len), int(max_seq_len)
+    a.ld_out, a.v_share = out.stride(0), v_share
     if long_min_q > 0 and long_stats is not None:
         a.long_min_q, (a.long_seqs, a.long_tokens, a.long_ctx_sum) = long_min_q, long_stats
     elif long_min_q > 0:
@@ -502,6 +506,46 @@ def delta_rule_scan(q, k, v, b_pre, a_pre, a_log, dt_bias, q_scale, state, state
     return _scan_common(a, q, k, v, state, state_slots, query_start, context_lens, H, G, dim, vdim)
 
 
+def ssm_scan(x, B, C_, dt_pre, a_log, dt_bias, skip, state, state_slots, query_start, context_lens, H, G, N, V):
+    """State-space recurrence over a mixed batch: x [T, H V], B, C_ [T, G N], dt_pre [T, H] -> float32 [T, H V]; state [slots, >= H N V]."""
+    from ._lib import StateScanArgs
+    a = StateScanArgs()
+    a.kind, a.a_pre, a.ld_a, a.a_log, a.dt_bias, a.skip, a.q_scale = 2, _p(dt_pre), dt_pre.stride(0), _p(a_log), _p(dt_bias), _p(skip), 1.0
+    return _scan_common(a, C_, B, x, state, state_slots, query_start, context_lens, H, G, N, V)
+
+
+def gate_groupnorm(o, gate, weight, parts, eps, out=None, zero_before=0, zero_after=0):
+    """o [T, n] float32; (o silu(gate)) RMS-normed in equal parts.  out: a view of n columns inside wider rows whose neighbouring columns
+    (zero_before in front, zero_after behind) are set to zero."""
+    T, n = o.shape
+    if out is None:
+        out = torch.empty((T, n), dtype=gate.dtype, device=o.device)
+    _lib.lib().atoma_gate_groupnorm(_p(o), _p(gate), gate.stride(0), _p(weight), _p(out), out.stride(0), T, n, parts, zero_before, zero_after, eps,
+                                    _CODES[gate.dtype], _s())
+    _check()
+    return out
+
+
+def differential_combine(maps, H, G, vdim, lam, gain, eps):
+    """maps [T, 2 H vdim] by groups (first map's heads, then the second's) -> [T, H vdim]."""
+    T = maps.shape[0]
+    out = torch.empty((T, H * vdim), dtype=maps.dtype, device=maps.device)
+    _lib.lib().atoma_differential_combine(_p(maps), _p(out), T, H, G, vdim, lam, gain, eps, _CODES[maps.dtype], _s())
+    _check()
+    return out
+
+
+def embed_pairs(tokens, token_seq, query_start, prev_tokens, table, pair_table, buckets, mul_prev, mul_cur, want_h=True):
+    """x [T, width] float32 and its copy in the table's format (or None)."""
+    T, W = tokens.shape[0], table.shape[1]
+    x = torch.empty((T, W), dtype=torch.float32, device=table.device)
+    h = torch.empty((T, W), dtype=table.dtype, device=table.device) if want_h else None
+    _lib.lib().atoma_embed_pairs(_p(tokens), _p(token_seq), _p(query_start), _p(prev_tokens), _p(table), _p(pair_table), buckets, mul_prev, mul_cur,
+                                 _p(x), _p(h), T, W, table.shape[0], _CODES[table.dtype], _s())
+    _check()
+    return x, h
+
+
 def headnorm_gate(o, weight, gate, H, vdim, eps, dtype):
     T = o.shape[0]
     out = torch.empty((T, H * vdim), dtype=dtype, device=o.device)
@@ -512,7 +556,7 @@ def headnorm_gate(o, weight, gate, H, vdim, eps, dtype):
 
 
 def qkv_headnorm_rope_cache(proj, q_off, k_off, v_off, q_w, k_w, qk_freq, v_freq, interleaved, positions, slots, k_cache, v_cache, H, G,
-                            dim, vdim, eps, bias=None, q_head_scale=None, unit_norm=False):
+                            dim, vdim, eps, bias=None, q_head_scale=None, unit_norm=False, qk_freq_lo=None, amplitude=1.0, v_heads=0):
     from ._lib import QkvRopeArgs
     T = proj.shape[0]
     q = torch.empty((T, H * dim), dtype=proj.dtype, device=proj.device)
@@ -523,6 +567,7 @@ def qkv_headnorm_rope_cache(proj, q_off, k_off, v_off, q_w, k_w, qk_freq, v_freq
     a.positions, a.slot_mapping, a.q_out, a.k_cache, a.v_cache = _p(positions), _p(slots), _p(q), _p(k_cache), _p(v_cache)
     a.T, a.H, a.G, a.dim, a.vdim, a.eps, a.dtype = T, H, G, dim, vdim, eps, _CODES[proj.dtype]
     a.bias, a.q_head_scale, a.unit_norm = _p(bias), _p(q_head_scale), int(unit_norm)
+    a.qk_freq_lo, a.qk_amplitude, a.v_heads = _p(qk_freq_lo), amplitude, v_heads
     _lib.lib().atoma_qkv_headnorm_rope_cache(C.byref(a), _s())
     _check()
     return q
@@ -565,9 +610,11 @@ def latent_expand_values(o_lat, w_uv, H, vdim, kv_rank, dtype, gate=None):
     return out
 
 
-def postnorm_residual(x, w_norm, alpha, eps, dtype, y=None, experts=None, depth=None, depth_w=None, depth_n=0, want_trace=False, offset=0.0):
+def postnorm_residual(x, w_norm, alpha, eps, dtype, y=None, experts=None, depth=None, depth_w=None, depth_n=0, want_trace=False, offset=0.0,
+                      branch_scale=None, y_bias=None, y_scale=1.0):
     """x [T, W] float32 is updated in place: x <- norm(alpha x + y + expert rows), row depth_n - 1 of depth [.., T, W] is written and x becomes
-    the weighted sum of its first depth_n rows.  experts: (expert_out address, pair_row address, top_expert, keep-alive).  Returns (h, trace)."""
+    the weighted sum of its first depth_n rows.  experts: (expert_out address, pair_row address, top_expert, keep-alive).
+    branch_scale: x <- alpha x + branch_scale norm(y_scale y + y_bias + expert rows) instead.  Returns (h, trace)."""
     from ._lib import PostnormArgs
     T, W = x.shape
     h = torch.empty((T, W), dtype=dtype, device=x.device)
@@ -577,6 +624,8 @@ def postnorm_residual(x, w_norm, alpha, eps, dtype, y=None, experts=None, depth=
     if experts is not None:
         a.expert_out, a.pair_row, a.top_expert, a.top = experts[0], experts[1], _p(experts[2]), experts[2].shape[1]
     a.T, a.width, a.alpha, a.eps, a.weight_offset, a.dtype = T, W, alpha, eps, offset, _CODES[dtype]
+    if branch_scale is not None:
+        a.norm_branch, a.branch_scale, a.y_bias, a.y_scale = 1, branch_scale, _p(y_bias), y_scale
     _lib.lib().atoma_postnorm_residual(C.byref(a), _s())
     _check()
     return h, trace
