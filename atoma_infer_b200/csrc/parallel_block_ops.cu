@@ -582,15 +582,12 @@ __device__ __forceinline__ void turn(float pos, float freq, float freq_lo, float
     cs = amplitude * fmaf(-rest, s, c * near_one);
 }
 
-// buf [n] float32 (one warp's): the first 2 pairs entries turned by pos * freq, written to dst as T.
+// buf [n] float32 (one warp's): the first 2 pairs entries turned by the token's angles (sin and cos of pair i at turns[2 i]), written to dst.
 template <typename T>
-__device__ __forceinline__ void rotate_store(const float *buf, int n, const float *__restrict__ freq, const float *__restrict__ freq_lo, float amplitude,
-                                             int pairs, int interleaved, float pos, T *__restrict__ dst, int lane) {
+__device__ __forceinline__ void rotate_store(const float *buf, int n, const float *turns, int pairs, int interleaved, T *__restrict__ dst, int lane) {
     for (int i = lane; i < pairs; i += 32) {
         const int ia = interleaved ? 2 * i : i, ib = interleaved ? 2 * i + 1 : i + pairs;
-        float sn, cs;
-        turn(pos, freq[i], freq_lo ? freq_lo[i] : 0.f, amplitude, sn, cs);
-        const float u = buf[ia], v = buf[ib];
+        const float sn = turns[2 * i], cs = turns[2 * i + 1], u = buf[ia], v = buf[ib];
         dst[ia] = from_f<T>(u * cs - v * sn);
         dst[ib] = from_f<T>(v * cs + u * sn);
     }
@@ -609,9 +606,15 @@ __global__ void __launch_bounds__(256) qkv_headnorm_rope_cache_kernel(const atom
     const int units = a.slot_mapping ? H + G + Gv : H;
     const float amplitude = a.qk_amplitude != 0.f ? a.qk_amplitude : 1.f;
     const int wide = max(D, V);
+    const int qk_pairs = a.qk_freq ? static_cast<int>(a.rot_pairs) : 0, v_pairs = a.v_freq ? static_cast<int>(a.v_pairs) : 0;
+    float *turns = sm + nwarp * wide, *v_turns = turns + 2 * qk_pairs;   // all heads of the token turn by the same angles
     float *buf = sm + warp * wide;
     const T *row = static_cast<const T *>(a.proj) + t * a.ld;
     const float pos = static_cast<float>(a.positions[t]);
+    for (int i = threadIdx.x; i < qk_pairs; i += blockDim.x)
+        turn(pos, a.qk_freq[i], a.qk_freq_lo ? a.qk_freq_lo[i] : 0.f, amplitude, turns[2 * i], turns[2 * i + 1]);
+    for (int i = threadIdx.x; i < v_pairs; i += blockDim.x) turn(pos, a.v_freq[i], 0.f, 1.f, v_turns[2 * i], v_turns[2 * i + 1]);
+    __syncthreads();
     const int64_t slot = a.slot_mapping ? a.slot_mapping[t] : -1;
     for (int u = warp; u < units; u += nwarp) {
         const bool is_q = u < H, is_k = !is_q && u < H + G;
@@ -639,9 +642,7 @@ __global__ void __launch_bounds__(256) qkv_headnorm_rope_cache_kernel(const atom
         T *dst = is_q ? static_cast<T *>(a.q_out) + (t * H + hd) * D
                       : (is_k ? static_cast<T *>(a.k_cache) + (slot * G + hd) * D : static_cast<T *>(a.v_cache) + (slot * Gv + hd) * V);
         const bool vpart = !is_q && !is_k;
-        const float *freq = vpart ? a.v_freq : a.qk_freq;
-        const int pairs = freq ? static_cast<int>(vpart ? a.v_pairs : a.rot_pairs) : 0;
-        rotate_store<T>(buf, n, freq, vpart ? nullptr : a.qk_freq_lo, vpart ? 1.f : amplitude, pairs, a.interleaved, pos, dst, lane);
+        rotate_store<T>(buf, n, vpart ? v_turns : turns, vpart ? v_pairs : qk_pairs, a.interleaved, dst, lane);
         __syncwarp();
     }
 }
@@ -890,7 +891,7 @@ bool hyb_qkv_headnorm_rope_cache(const atoma_qkv_rope_args &a, cudaStream_t stre
         return false;
     }
     const unsigned warps = static_cast<unsigned>(std::min<int64_t>(8, a.H + 2 * a.G));
-    const size_t smem = static_cast<size_t>(warps) * std::max(a.dim, a.vdim) * 4;
+    const size_t smem = (static_cast<size_t>(warps) * std::max(a.dim, a.vdim) + 2 * (a.rot_pairs + a.v_pairs)) * 4;
     if (smem > 48 * 1024) {
         set_status(kErrUnsupported, "atoma_qkv_headnorm_rope_cache: heads of %lld entries", static_cast<long long>(std::max(a.dim, a.vdim)));
         return false;
