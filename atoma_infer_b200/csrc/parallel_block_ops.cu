@@ -5,7 +5,7 @@
 // layer and with its input norm).  The mixers that need more than attention kernels:
 //   - tap filters whose inputs before a portion come from a per-sequence history (the portion's last inputs replace it),
 //   - matrix-state recurrences (gated linear attention, gated delta rule, state-space recurrence): every head keeps S [dim, vdim] in float32; the
-//     columns of S are independent in both recurrences, so a CTA owns 32 columns of one head of one sequence, the rows
+//     columns of S are independent in all of them, so a CTA owns 32 columns of one head of one sequence, the rows
 //     of a column are spread over `parts` threads (registers), and the tokens are visited strictly in order,
 //   - rotary positions on queries, keys and values with the cache write, the turn-back of a head's sum, and the
 //     latent-attention variants that keep one rotated key part beside the latent.
