@@ -22,10 +22,10 @@ from bench_mobunex import _serve
 from bench_patadra import _row
 
 SIZES = {
-    "2k-wide": dict(width=2048, vocab=32000, ff=8192, window=1024, mult=0.7, attention=dict(heads=16, kv_heads=4, dim=64, vdim=128, rot=32),
+    "2k-wide": dict(width=2048, vocab=32000, ff=8192, window=1024, mult=0.9, attention=dict(heads=16, kv_heads=4, dim=64, vdim=128, rot=32),
                     left=dict(heads=32, kv_heads=8, dim=64, vdim=64, rot=64), right=dict(heads=32, vdim=64, groups=8, state=128, norm_groups=8, taps=4),
                     layers=("parallel", "attention", "parallel", "shared")),
-    "4k-wide": dict(width=4096, vocab=32000, ff=14336, window=4096, mult=0.7, attention=dict(heads=32, kv_heads=8, dim=64, vdim=128, rot=32),
+    "4k-wide": dict(width=4096, vocab=32000, ff=14336, window=4096, mult=0.9, attention=dict(heads=32, kv_heads=8, dim=64, vdim=128, rot=32),
                     left=dict(heads=32, kv_heads=8, dim=128, vdim=128, rot=128), right=dict(heads=64, vdim=64, groups=8, state=128, norm_groups=8, taps=4),
                     layers=("parallel", "attention", "parallel", "shared")),
 }
@@ -37,10 +37,10 @@ def _spec(s):
     source = s["layers"].index("attention")
     attn = lambda kv_from: dict(mixer="softmax_attention",
                                 softmax=SoftmaxAttentionSpec(a["heads"], a["kv_heads"], a["dim"], a["vdim"], 1 / math.sqrt(a["dim"]), s["window"], bias=True, qk_norm=True,
-                                                             rotary=RotarySpec(a["rot"], 5e5), out_bias=True, maps=2, diff=0.3, kv_from=kv_from))
+                                                             rotary=RotarySpec(a["rot"], 1e5), out_bias=True, maps=2, diff=0.4, kv_from=kv_from))
     both = MixerSumSpec(SoftmaxAttentionSpec(l["heads"], l["kv_heads"], l["dim"], l["vdim"], 1 / math.sqrt(l["dim"]), qk_norm=True,
-                                             rotary=RotarySpec(l["rot"], 1e6, yarn=(4.0, 2048, 32.0, 1.0))),
-                        StateSpaceSpec(d["heads"], d["vdim"], d["groups"], d["state"], d["norm_groups"], d["taps"]), 0.6, 1.1)
+                                             rotary=RotarySpec(l["rot"], 5e5, yarn=(4.0, 2048, 32.0, 1.0))),
+                        StateSpaceSpec(d["heads"], d["vdim"], d["groups"], d["state"], d["norm_groups"], d["taps"]), 0.8, 1.25)
     mixers = {"attention": attn(None), "shared": attn(source), "parallel": dict(mixer="attention_ssm", mixer_sum=both)}
     return HybridSpec(s["width"], s["vocab"], 1e-5, 1.0, tuple(LayerSpec(mlp=MlpSpec(s["ff"], "silu"), **mixers[k]) for k in s["layers"]), norm_offset=1.0,
                       block_style="postnorm", position="none", embed_norm=False, branch_scale=s["mult"], pair_table=PairTableSpec(30011, 1019, 31))
@@ -122,7 +122,7 @@ def _kernel_rows(torch, s, dev, steps, warmup, hbm, tf):
         attention("mobunex_softmax_attention_128", H // 2, G // 2, 1, V, V, win)          # as many value bytes
         attention("left_attention", l["heads"], l["kv_heads"], 1, l["dim"], l["vdim"], 0)
         maps = rn(T, H * V)
-        put(f"differential_combine_{name}", lambda: ho.differential_combine(maps, H // 2, G // 2, V, 0.4, 0.7, 1e-5), nbytes=T * H * V * 3)
+        put(f"differential_combine_{name}", lambda: ho.differential_combine(maps, H // 2, G // 2, V, 0.4, 0.6, 1e-5), nbytes=T * H * V * 3)
         del maps
         torch.cuda.empty_cache()
         # ---- the recurrence beside the attention ----
@@ -154,7 +154,7 @@ def _kernel_rows(torch, s, dev, steps, warmup, hbm, tf):
     # ---- row operators at 8192 tokens ----
     T = 8192
     x, y, wn = torch.randn((T, W), device=dev), rn(T, W), torch.ones(W, device=dev)
-    put("branch_norm_update", lambda: ho.postnorm_residual(x, wn, 1.0, 1e-5, bf, y=y, offset=1.0, branch_scale=0.7, y_bias=wn), nbytes=T * W * (8 + 2 + 2))
+    put("branch_norm_update", lambda: ho.postnorm_residual(x, wn, 1.0, 1e-5, bf, y=y, offset=1.0, branch_scale=0.9, y_bias=wn), nbytes=T * W * (8 + 2 + 2))
     put("mobunex_postnorm_residual", lambda: ho.postnorm_residual(x, wn, 2.0, 1e-5, bf, y=y), nbytes=T * W * (8 + 2 + 2))
     toks, tseq, qs = torch.randint(0, s["vocab"], (T,), device=dev, dtype=torch.int32), torch.zeros(T, device=dev, dtype=torch.int32), i32([0, T])
     table, pairs = rn(s["vocab"], W), rn(30012, W)

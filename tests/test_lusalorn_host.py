@@ -82,7 +82,7 @@ def test_what_the_design_does_not_have_is_refused():
 
 
 def test_yarn_frequencies_follow_the_rule():
-    for dims, base, sc in ((24, 30000.0, dict(factor=6.0, original=2048, fast=24.0, slow=1.5)), (48, 1e6, dict(factor=3.0, original=512, fast=32.0, slow=1.0)), (12, 500.0, None)):
+    for dims, base, sc in ((24, 30000.0, dict(factor=6.0, original=2048, fast=24.0, slow=1.5)), (44, 2e5, dict(factor=3.0, original=512, fast=32.0, slow=1.0)), (12, 500.0, None)):
         f, amp = lo.rotary_frequencies(dict(dims=dims, base=base, scaling=sc))
         r = RotarySpec(dims=dims, base=base, yarn=None if sc is None else tuple(sc[k] for k in ("factor", "original", "fast", "slow")))
         assert abs(r.amplitude - amp) < 1e-15
